@@ -1,11 +1,11 @@
 """Host-side bookkeeping of the paged cache: pools, groups, block tables, slots.
 
 Keys and values live in fixed-size pages.  Layers with the same needs (all keys, or a
-window of them, for a given head geometry) form a *group* with a pool and a block table of
+window or chunk of them, for a given head geometry) form a *group* with a pool and a block table of
 its own; every layer of a group uses the same page ids.  A request holds a *slot* (its row
 in every block table and in every per-request state tensor) and, per group, a list of
-pages.  Pages go back to the pool when the request ends, or, in a windowed group, as soon
-as the window has passed them; they are handed out again to whoever asks next.
+pages.  Pages go back to the pool when the request ends, or, in a windowed or chunked group, as
+soon as the window or the chunk has passed them; they are handed out again to whoever asks next.
 
 The reference keeps the same bookkeeping in ``BlockPool`` (null block 0, all-or-nothing
 ``get_new_blocks``, freed blocks reused first: ``rapid_llm/engine/block_pool.py:156-303``),
@@ -99,7 +99,16 @@ class GroupSpec:
 
     @property
     def window(self) -> int:
+        """Most positions a query sees, its own included (a window, a chunk); 0 = every one before it."""
+        if self.need.kind == "chunk":
+            return self.need.chunk
         return self.need.window if self.need.kind == "window" else 0
+
+    def oldest_visible(self, position: int) -> int:
+        """The first position that a query at ``position``, or any later one, can see."""
+        if self.need.kind == "chunk":
+            return position - position % self.need.chunk
+        return max(position - self.window + 1, 0) if self.window else 0
 
 
 def plan_groups(needs: Sequence[CacheNeed | None]) -> tuple[list[GroupSpec], list[int | None]]:
@@ -112,10 +121,12 @@ def plan_groups(needs: Sequence[CacheNeed | None]) -> tuple[list[GroupSpec], lis
         if need is None:
             entry_group.append(None)
             continue
-        if need.kind not in ("full", "window"):
+        if need.kind not in ("full", "window", "chunk"):
             raise ValueError(f"unknown cache kind {need.kind!r}")
         if need.kind == "window" and need.window < 1:
             raise ValueError("a windowed cache needs window >= 1")
+        if need.kind == "chunk" and need.chunk < 1:
+            raise ValueError("a cache of chunks needs chunk >= 1")
         if need.elements_per_token() < 1:
             raise ValueError("a cache need must give kv heads and a head size, or the shape of a token's row")
         key = need.group_key()
@@ -246,20 +257,18 @@ class CacheManager:
         return True
 
     def release_passed(self, request_id: Hashable) -> int:
-        """Free the pages of windowed groups that no later query can reach.
+        """Free the pages of windowed and chunked groups that no later query can reach.
 
         The next query sits at position ``num_tokens`` and reaches back to
-        ``num_tokens - window + 1``; pages wholly below that are dead.  Returns how many
-        pages were given back.
+        ``num_tokens - window + 1``, or to the start of its chunk; pages wholly below that are
+        dead.  Returns how many pages were given back.
         """
         held = self._get(request_id)
         released = 0
         for index, group in enumerate(self.groups):
-            window = group.window
-            if not window:
+            if not group.window:
                 continue
-            oldest = max(held.num_tokens - window + 1, 0)
-            keep_from = min(oldest // self.page_size, len(held.pages[index]))
+            keep_from = min(group.oldest_visible(held.num_tokens) // self.page_size, len(held.pages[index]))
             dead = [page for page in held.pages[index][:keep_from] if page != NULL_PAGE]
             if not dead:
                 continue

@@ -3,6 +3,7 @@
 from .engine_config import EngineConfig, parse_dtype
 from .model_spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
 from .basitar import BasitarConfig
+from .bidetar import BidetarConfig
 from .kopatar import KopatarConfig
 from .mezadra import MezadraConfig
 from .qwen3 import Qwen3Config
@@ -20,9 +21,11 @@ register_architecture(KopatarConfig)
 register_architecture(MezadraConfig)
 register_architecture(BasitarConfig)
 register_architecture(ZupupelConfig)
+register_architecture(BidetarConfig)
 
 __all__ = [
     "BasitarConfig",
+    "BidetarConfig",
     "EngineConfig",
     "KopatarConfig",
     "LayerSpec",

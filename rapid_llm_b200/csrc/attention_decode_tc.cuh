@@ -28,7 +28,7 @@
 //     through distributed shared memory, in rank order: no scratch in global memory and no
 //     second kernel.
 //
-// Semantics are those of attention_mma.cu (scores, running maximum and sum and the output
+// Semantics are those of attention_mma.cu, a sink and chunks included, squashed scores not (scores, running maximum and sum and the output
 // accumulator in float32; P rounded to bfloat16 before P.V).  Needs head size 128 and pages of
 // 8, 16, 32, 64 or a multiple of 128 tokens; everything else takes the mma.sync kernel.
 #pragma once
@@ -73,9 +73,10 @@ struct DecodeTcArgs {
   const int* entry_start;
   const int* entry_slot;
   const int* block_table;
-  int hq, hkv, page_size, num_pages, max_pages, slots, window, splits;
+  int hq, hkv, page_size, num_pages, max_pages, slots, window, chunk, splits;
   int cluster_merge;        // the CTAs of an item's splits are one cluster and merge among themselves
   float scale_log2;
+  const float* sink;        // [hq] float32 or null: exp(sink[head]) joins every row's denominator once
   int* fault;
 };
 
@@ -131,7 +132,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
   if (bad && tid == 0)
     atomicOr(args.fault, (slot < 0 || slot >= args.slots) ? kFaultSlot : kFaultPosition);
   const int hi = bad ? 0 : max_pos + 1;
-  const int lo = args.window > 0 ? max(0, min_pos - args.window + 1) : 0;
+  const int lo = first_visible(min_pos, args.window, args.chunk);
   const int lo_aligned = lo & ~(kTcKeys - 1);
   const int span = max(hi - lo_aligned, 0);
   const int per_split = ((span + args.splits - 1) / args.splits + kTcKeys - 1) / kTcKeys * kTcKeys;
@@ -168,7 +169,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
     const int p = row0 + tid;
     const int pos = tid < n_rows ? start + p / group : -1;       // -1: a row that sees no key
     row_pos[tid] = pos;
-    row_lo[tid] = args.window > 0 ? max(0, pos - args.window + 1) : 0;
+    row_lo[tid] = first_visible(pos, args.window, args.chunk);
   }
   // the page ids of this item's key range (the block table is complete before the step starts)
   const int first_page = k_begin / args.page_size;
@@ -471,11 +472,18 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
       const float w0 = fast_exp2(run_max[n] - safe), w1 = fast_exp2(max1 - safe);
       const float total = sum0 * w0 + sum1 * w1;
       const float value = out_acc[n] * w0 + exchange[n * 128 + t] * w1;
-      const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+      float inv = total > 0.0f ? 1.0f / total : 0.0f;
       const float lse = total > 0.0f ? m + log2f(total) : -INFINITY;
-      const float merged = value * inv;
       const int p = row0 + n, token = p / group;
       const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group + (p - token * group);
+      if (args.sink != nullptr && args.splits == 1) {
+        // an unsplit row's denominator takes the sink here; a split one's where its parts meet
+        const float sink2 = args.sink[row % args.hq] * 1.4426950408889634f;
+        const float top = fmaxf(m, sink2);
+        const float keys = m == -INFINITY ? 0.0f : fast_exp2(m - top);
+        inv = keys / (total * keys + fast_exp2(sink2 - top));
+      }
+      const float merged = value * inv;
       if (args.splits == 1) {
         args.out[row * kTcD + t] = __float2bfloat16_rn(merged);
       } else if (args.cluster_merge) {
@@ -523,7 +531,10 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
             }
           }
         }
-        float m = -INFINITY;
+        const int p = row0 + n, token = p / group;
+        const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group + (p - token * group);
+        const float sink2 = args.sink != nullptr ? args.sink[row % args.hq] * 1.4426950408889634f : -INFINITY;
+        float m = sink2;
 #pragma unroll
         for (int r = 0; r < 8; ++r) m = fmaxf(m, lse_of[r]);
         if (wide) {
@@ -531,7 +542,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
           for (int r = 8; r < kTcMaxClusterSplits; ++r) m = fmaxf(m, lse_of[r]);
         }
         const float safe = m == -INFINITY ? 0.0f : m;
-        float total = 0.0f, value = 0.0f;
+        float total = args.sink != nullptr ? fast_exp2(sink2 - safe) : 0.0f, value = 0.0f;
 #pragma unroll
         for (int r = 0; r < 8; ++r) {
           if (r < args.splits) {
@@ -550,8 +561,6 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
             }
           }
         }
-        const int p = row0 + n, token = p / group;
-        const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group + (p - token * group);
         args.out[row * kTcD + t] = __float2bfloat16_rn(total > 0.0f ? value / total : 0.0f);
       }
     }

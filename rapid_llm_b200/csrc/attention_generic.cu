@@ -1,6 +1,6 @@
 // Paged causal attention for any head size (steps of 16 up to 256; up to 640 in a second build of the
 // kernel with more registers, for cached latent rows wider than the tensor-core tiles take), any number of heads
-// and groups, any page size, with an optional window; one warp per (token, query head).
+// and groups, any page size, with an optional window or chunks; one warp per (token, query head).
 //
 // This is the kernel of the float32 path and the fallback of the bfloat16 path for head
 // sizes the tensor-core kernels are not instantiated for.  Every token of the step is a
@@ -12,7 +12,7 @@
 // rapid_llm/kernels/ops/attention/flashdecoding.py:223-230): kv head = q head // group;
 // s_j = (q . k_j) * scale over the cached positions j <= p of the same request (and
 // j > p - window when a window is set: the query's own position counts, as in
-// rapid_llm/engine/kv_cache_spec.py:204,221-224); softmax over j; o = sum_j P_j v_j.
+// rapid_llm/engine/kv_cache_spec.py:204,221-224; and j of the chunk p lies in when a chunk size is set); softmax over j; o = sum_j P_j v_j.
 // Scores, running maximum and sum, and the output accumulator are float32.
 #include "common.cuh"
 
@@ -31,7 +31,7 @@ __global__ void attention_generic_kernel(
     const int* __restrict__ token_slot, // [tokens]
     const int* __restrict__ block_table,  // [slots, max_pages]
     int tokens, int hq, int hkv, int d, int page_size, int num_pages, int max_pages, int slots,
-    int window, float scale, float softcap, const float* __restrict__ sink, int kv_planes, int* __restrict__ fault) {
+    int window, int chunk, float scale, float softcap, const float* __restrict__ sink, int kv_planes, int* __restrict__ fault) {
   __shared__ float q_staged[kGenericWarps][kMaxD];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = static_cast<long long>(blockIdx.x) * kGenericWarps + warp;
@@ -54,7 +54,7 @@ __global__ void attention_generic_kernel(
   for (int i = lane; i < d; i += 32) qs[i] = to_float(qr[i]) * scale;
   __syncwarp();
 
-  const int first = window > 0 ? max(0, pos - window + 1) : 0;
+  const int first = first_visible(pos, window, chunk);
   const size_t head_stride = static_cast<size_t>(page_size) * d;
   // K plane -> V plane; a cache of one plane keeps rows that are keys and values at once
   const size_t v_offset = kv_planes == 2 ? static_cast<size_t>(hkv) * head_stride : 0;
@@ -131,11 +131,11 @@ extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache,
                                     const int* positions, const int* token_slot,
                                     const int* block_table, int tokens, int hq, int hkv, int d,
                                     int page_size, int num_pages, int max_pages, int slots,
-                                    int window, float scale, float softcap, const float* sink, int kv_planes,
+                                    int window, int chunk, float scale, float softcap, const float* sink, int kv_planes,
                                     int* fault, cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (d <= 0 || d % 16 != 0 || d > rl::kGenericWideD || hkv <= 0 || hq % hkv != 0 ||
-      page_size <= 0 || window < 0 || softcap < 0.0f || kv_planes < 1 || kv_planes > 2)
+      page_size <= 0 || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || softcap < 0.0f || kv_planes < 1 || kv_planes > 2)
     return static_cast<int>(cudaErrorInvalidValue);
   const long long items = static_cast<long long>(tokens) * hq;
   const unsigned blocks =
@@ -146,7 +146,7 @@ extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache,
     kernel<<<blocks, rl::kGenericWarps * 32, 0, stream>>>(
         static_cast<const scalar_t*>(q), static_cast<const scalar_t*>(cache),
         static_cast<scalar_t*>(out), positions, token_slot, block_table, tokens, hq, hkv, d,
-        page_size, num_pages, max_pages, slots, window, scale, softcap, sink, kv_planes, fault);
+        page_size, num_pages, max_pages, slots, window, chunk, scale, softcap, sink, kv_planes, fault);
   });
   return rl::launch_status();
 }

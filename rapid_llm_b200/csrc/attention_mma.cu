@@ -18,7 +18,7 @@
 // Formula (rapid_llm/kernels/ops/attention/flashattention2_nopad.py:85,141-168,
 // rapid_llm/kernels/ops/attention/flashdecoding.py:223-230,335-407): kv head = q head //
 // group; s_j = (q . k_j) * scale for cached j <= p of the same request (and j > p - window
-// when a window is set); softmax over j; o = sum_j P_j v_j.  Scores, running maximum and
+// when a window is set; j of p's own chunk when a chunk size is set); softmax over j; o = sum_j P_j v_j.  Scores, running maximum and
 // sum and the output accumulator are float32; the exponent is taken in base 2 with log2(e)
 // folded into the scale; P is rounded to bfloat16 before the P.V product, as the
 // reference's tensor-core kernels do (flashattention2_nopad.py:162).
@@ -63,10 +63,10 @@ struct AttentionArgs {
   const int* entry_start;   // [entries]  tokens cached before this step
   const int* entry_slot;    // [entries]
   const int* block_table;   // [slots, max_pages]
-  int hq, hkv, page_size, num_pages, max_pages, slots, window, splits;
+  int hq, hkv, page_size, num_pages, max_pages, slots, window, chunk, splits;   // a window, a chunk size, or neither
   float scale_log2;         // scale * log2(e)
   int* fault;
-  // Squashed scores and a sink (the mma.sync tiles, the merge kernel and the tcgen05 chunk tiles; not the tcgen05 decode tiles):
+  // Squashed scores (the mma.sync tiles and the tcgen05 chunk tiles; not the tcgen05 decode tiles) and a sink (all tiles and the merge kernel):
   // with softcap > 0 a score s becomes softcap * tanh(s / softcap) after the scale; with `sink` ([hq], float32)
   // every row's denominator also holds exp(sink[head]), a term without a key or a value, counted once.
   float scale;              // the plain scale (used with softcap)
@@ -151,7 +151,7 @@ attention_mma_kernel(const AttentionArgs args) {
     row_token[i] = tok_begin + token;
     row_head[i] = kv_head * group + (p - token * group);
     row_pos[i] = row_valid[i] ? start + token : -1;
-    row_lo[i] = args.window > 0 ? max(0, row_pos[i] - args.window + 1) : 0;
+    row_lo[i] = first_visible(row_pos[i], args.window, args.chunk);
   }
 
   const int last_row = min(n_rows, row0 + kTileM) - 1;
@@ -163,7 +163,7 @@ attention_mma_kernel(const AttentionArgs args) {
   }
   // key range of the tile, then of this split (begin on a multiple of 64)
   const int hi = bad ? 0 : max_pos + 1;
-  const int lo = args.window > 0 ? max(0, min_pos - args.window + 1) : 0;
+  const int lo = first_visible(min_pos, args.window, args.chunk);
   const int lo_aligned = lo & ~(kBlockN - 1);
   const int span = max(hi - lo_aligned, 0);
   const int per_split = ((span + args.splits - 1) / args.splits + kBlockN - 1) / kBlockN * kBlockN;
@@ -583,7 +583,7 @@ static int launch_prefill_tc(const AttentionArgs& a, int n_items, bool pdl, cuda
   t.q = a.q; t.out = a.out; t.items = a.items; t.cu_seqlens = a.cu_seqlens; t.entry_start = a.entry_start;
   t.entry_slot = a.entry_slot; t.block_table = a.block_table; t.hq = a.hq; t.hkv = a.hkv;
   t.page_size = a.page_size; t.num_pages = a.num_pages; t.max_pages = a.max_pages; t.slots = a.slots;
-  t.window = a.window; t.scale_log2 = a.scale_log2; t.fault = a.fault;
+  t.window = a.window; t.chunk = a.chunk; t.scale_log2 = a.scale_log2; t.fault = a.fault;
   t.softcap = a.softcap; t.sink = a.sink; t.cap_in = 0.0f; t.cap_out = 0.0f;
   if (a.softcap > 0.0f) {
     t.cap_in = 2.0f * 1.4426950408889634f * a.scale / a.softcap;
@@ -671,7 +671,7 @@ static int launch_decode_tc(const AttentionArgs& a, int n_items, int max_rows, b
   t.cu_seqlens = a.cu_seqlens; t.entry_start = a.entry_start; t.entry_slot = a.entry_slot;
   t.block_table = a.block_table; t.hq = a.hq; t.hkv = a.hkv; t.page_size = a.page_size;
   t.num_pages = a.num_pages; t.max_pages = a.max_pages; t.slots = a.slots; t.window = a.window;
-  t.splits = a.splits; t.cluster_merge = cluster_merge ? 1 : 0; t.scale_log2 = a.scale_log2; t.fault = a.fault;
+  t.chunk = a.chunk; t.sink = a.sink; t.splits = a.splits; t.cluster_merge = cluster_merge ? 1 : 0; t.scale_log2 = a.scale_log2; t.fault = a.fault;
   if (max_rows <= 0 || max_rows > kTcRows) max_rows = kTcRows;
   if (max_rows <= 1) return launch_decode_tc_rows<1>(map, t, n_items, pdl, stream, g_decode_tc_configured[0], rings);
   if (max_rows <= 2) return launch_decode_tc_rows<2>(map, t, n_items, pdl, stream, g_decode_tc_configured[1], rings);
@@ -736,13 +736,12 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
                      int n_decode_items, const int* cu_seqlens, const int* entry_start,
                      const int* entry_slot, const int* block_table, int tokens, int hq, int hkv,
                      int head_dim, int page_size, int num_pages, int max_pages, int slots,
-                     int window, int splits, float scale, int* fault, int pdl, int decode_kernel, int decode_rows,
+                     int window, int chunk, int splits, float scale, int* fault, int pdl, int decode_kernel, int decode_rows,
                      int chunk_rows, int decode_splits, float softcap, const float* sink, int kv_planes,
                      cudaStream_t stream) {
   if (tokens == 0 || (n_chunk_items == 0 && n_decode_items == 0)) return 0;
-  const bool plain_scores = !(softcap > 0.0f) && sink == nullptr;
-  if (!plain_scores) {          // squashed scores and sinks: the tcgen05 chunk tiles and the mma.sync tiles take them
-    if (softcap < 0.0f || (decode_splits > 0 && decode_splits != splits)) return static_cast<int>(cudaErrorInvalidValue);
+  if (softcap != 0.0f) {        // squashed scores: the tcgen05 chunk tiles and the mma.sync tiles take them
+    if (!(softcap > 0.0f) || (decode_splits > 0 && decode_splits != splits)) return static_cast<int>(cudaErrorInvalidValue);
     decode_kernel = 1;
   }
   if (kv_planes == 1) {         // rows that are keys and values at once: the mma.sync tiles read them, the tcgen05 tiles do not
@@ -752,7 +751,7 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
     return static_cast<int>(cudaErrorInvalidValue);
   }
   if (head_dim != attn::kD || hkv <= 0 || hq % hkv != 0 || page_size <= 0 || window < 0 ||
-      splits < 1 || (splits > 1 && (part_out == nullptr || part_lse == nullptr)) ||
+      chunk < 0 || (window > 0 && chunk > 0) || splits < 1 || (splits > 1 && (part_out == nullptr || part_lse == nullptr)) ||
       hkv > 65535 || n_chunk_items > 65535 || n_decode_items > 65535)      // grid y dimensions
     return static_cast<int>(cudaErrorInvalidValue);
   // key ranges of the decode tiles alone (0 = as `splits`): only where the chunk tiles are not split and the decode
@@ -772,7 +771,7 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
   args.entry_slot = entry_slot;
   args.block_table = block_table;
   args.hq = hq; args.hkv = hkv; args.page_size = page_size; args.num_pages = num_pages;
-  args.max_pages = max_pages; args.slots = slots; args.window = window; args.splits = splits;
+  args.max_pages = max_pages; args.slots = slots; args.window = window; args.chunk = chunk; args.splits = splits;
   args.scale_log2 = scale * 1.4426950408889634f;
   args.fault = fault;
   args.scale = scale; args.softcap = softcap; args.sink = sink; args.kv_planes = kv_planes;
@@ -901,7 +900,7 @@ int rl_attention_mma_static_scratch(const void* q, const void* cache, void* out,
   }
   return rl_attention_mma(q, cache, out, part_out, part_lse, chunk_items, n_chunk_items, decode_items,
                           n_decode_items, cu_seqlens, entry_start, entry_slot, block_table, tokens, hq, hkv,
-                          head_dim, page_size, num_pages, max_pages, slots, window, splits, scale, fault, 0, 1, 0, 64, 0, 0.0f, nullptr, 2, stream);
+                          head_dim, page_size, num_pages, max_pages, slots, window, 0, splits, scale, fault, 0, 1, 0, 64, 0, 0.0f, nullptr, 2, stream);
 }
 
 }  // extern "C"

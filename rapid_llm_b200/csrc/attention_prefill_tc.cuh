@@ -88,7 +88,7 @@ struct PrefillTcArgs {
   const int* entry_start;
   const int* entry_slot;
   const int* block_table;
-  int hq, hkv, page_size, num_pages, max_pages, slots, window;
+  int hq, hkv, page_size, num_pages, max_pages, slots, window, chunk;
   float scale_log2;
   int* fault;
   // Squashed scores (softcap > 0: a scaled score s becomes softcap * tanh(s / softcap)) and a sink ([hq] float32 or
@@ -141,7 +141,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const
   if (bad && tid == 0)
     atomicOr(args.fault, (slot < 0 || slot >= args.slots) ? kFaultSlot : kFaultPosition);
   const int hi = bad ? 0 : max_pos + 1;
-  const int lo = args.window > 0 ? max(0, min_pos - args.window + 1) : 0;
+  const int lo = first_visible(min_pos, args.window, args.chunk);
   const int k_begin = lo & ~(kPfKeys - 1);
   const int n_blocks = hi > k_begin ? (hi - k_begin + kPfKeys - 1) / kPfKeys : 0;
   // blocks each tile needs: up to its last row's position
@@ -333,7 +333,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const
     const bool valid = p < row0 + n_rows && !bad;
     const int token = p / group;
     const int pos = valid ? start + token : -1;        // -1: a row that sees no key
-    const int lo_pos = args.window > 0 ? max(0, pos - args.window + 1) : 0;
+    const int lo_pos = first_visible(pos, args.window, args.chunk);
     pdl_wait();                                        // queries come from the kernel before
     {
       // The warp's 32 rows of Q, 256 bytes each, into the K-major operand [row][64] x 2 halves, swizzled: an

@@ -101,6 +101,15 @@ __device__ __forceinline__ int entry_of(const int* __restrict__ cu_seqlens, int 
   return lo;
 }
 
+// The first key position a query at `pos` sees: with a window the last `window` positions (its own included), with a
+// chunk size the positions from the start of its own chunk, chunks being counted from position 0 of the sequence
+// (one of the two at most; neither: every position from 0).  A row that sees no key has pos = -1 and gets 0.
+__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
+  if (pos < 0) return 0;
+  if (chunk > 0) return pos - pos % chunk;
+  return window > 0 ? max(0, pos - window + 1) : 0;
+}
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // ---- programmatic dependent launch -------------------------------------------------------

@@ -126,7 +126,7 @@ __global__ void embedding_sum_kernel(T* __restrict__ out, float* __restrict__ st
 // One block per output row.  Row i of the output reads input row `row_index[i]`
 // (or i when row_index is null).
 //   mode 0: r = x                 (first layer: the residual stream starts here)
-//   mode 1: r = x + residual
+//   mode 1: r = x_scale * x + residual (x_scale weighs what a sublayer adds to the stream)
 //   mode 2: r = x, residual untouched and may be null (a plain norm)
 //   mode 3: r = residual, x unread (the norm of the stream itself, for models whose sublayers add
 //           their normed outputs to it)
@@ -148,7 +148,7 @@ template <typename TX, typename TOut, bool kVector>
 __global__ void add_rmsnorm_kernel(const TX* __restrict__ x, float* __restrict__ residual,
                                    const float* __restrict__ weight, TOut* __restrict__ out,
                                    const int* __restrict__ row_index, int hidden, float eps,
-                                   int mode, int write_residual, const TX* extra_rows,
+                                   int mode, int write_residual, float x_scale, const TX* extra_rows,
                                    const float* __restrict__ extra_vector) {
   extern __shared__ float row_values[];  // [hidden] on the element-by-element path
   __shared__ float scratch[32];
@@ -173,7 +173,7 @@ __global__ void add_rmsnorm_kernel(const TX* __restrict__ x, float* __restrict__
         float r[8];
         load8(rr + at, r);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) v[i] += r[i];
+        for (int i = 0; i < 8; ++i) v[i] = fmaf(x_scale, v[i], r[i]);
       }
       if (er) {
         float extra[8];
@@ -225,7 +225,7 @@ __global__ void add_rmsnorm_kernel(const TX* __restrict__ x, float* __restrict__
     float sum_sq = 0.0f;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
       float v = mode == 3 ? rr[i] : to_float(xr[i]);
-      if (mode == 1) v += rr[i];
+      if (mode == 1) v = fmaf(x_scale, v, rr[i]);
       if (er) v += to_float(er[i]);
       if (extra_vector && mode != 5) v += extra_vector[i];
       if (write_residual && mode < 4) rr[i] = v;
@@ -341,12 +341,13 @@ __global__ void layernorm_kernel(const T* __restrict__ x, float* __restrict__ re
   }
 }
 
-// ------------------------------------------------------------ a sigmoid gate, entry by entry
-// out[t, c] = rows[t, c] * sigmoid(gate[t, c]), float32 arithmetic, one rounding; `gate` may be a view of some
-// columns of wider rows (gate_stride).  kVector: eight entries (16 bytes of bfloat16) a thread and step.
+// ------------------------------------------------------------ a sigmoid gate, entry by entry or one number a head
+// out[t, c] = rows[t, c] * sigmoid(gate[t, c / per]), float32 arithmetic, one rounding; `per` 1: a number an entry,
+// or the head size: a number a head.  `gate` and `out` may be views of some columns of wider rows (their strides), and
+// of the same rows (not of the same columns).  kVector: eight entries (16 bytes of bfloat16) a thread and step.
 template <typename T, bool kVector>
-__global__ void sigmoid_gate_kernel(const T* __restrict__ rows, const T* __restrict__ gate, int gate_stride,
-                                    T* __restrict__ out, int tokens, int width) {
+__global__ void sigmoid_gate_kernel(const T* __restrict__ rows, const T* gate, int gate_stride,
+                                    T* out, int out_stride, int tokens, int width, int per) {
   pdl_trigger();
   pdl_wait();
   constexpr int kStep = kVector ? 8 : 1;
@@ -359,13 +360,48 @@ __global__ void sigmoid_gate_kernel(const T* __restrict__ rows, const T* __restr
     if constexpr (kVector) {
       float v[8], g[8];
       load8(rows + t * width + c, v);
-      load8(gate + t * gate_stride + c, g);
+      if (per > 1) {       // a head's size is a multiple of eight here: the eight entries share their number
+        const float factor = 1.0f / (1.0f + expf(-to_float(gate[t * gate_stride + c / per])));
 #pragma unroll
-      for (int i = 0; i < 8; ++i) v[i] = v[i] / (1.0f + expf(-g[i]));
-      store8(out + t * width + c, v);
+        for (int i = 0; i < 8; ++i) v[i] *= factor;
+      } else {
+        load8(gate + t * gate_stride + c, g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = v[i] / (1.0f + expf(-g[i]));
+      }
+      store8(out + t * out_stride + c, v);
     } else {
-      const float g = to_float(gate[t * gate_stride + c]);
-      out[t * width + c] = from_float<T>(to_float(rows[t * width + c]) / (1.0f + expf(-g)));
+      const float g = to_float(gate[t * gate_stride + c / per]);
+      out[t * out_stride + c] = from_float<T>(to_float(rows[t * width + c]) / (1.0f + expf(-g)));
+    }
+  }
+}
+
+// ------------------------------------------------------------ the square of relu
+// out[t, c] = max(in[t, c], 0)^2 (float32 arithmetic); both may be views of some columns of wider rows, and the same one.
+template <typename T, bool kVector>
+__global__ void relu_squared_kernel(const T* in, int in_stride, T* out, int out_stride, int tokens, int width) {
+  pdl_trigger();
+  pdl_wait();
+  constexpr int kStep = kVector ? 8 : 1;
+  const size_t per_row = static_cast<size_t>(width / kStep);
+  const size_t total = static_cast<size_t>(tokens) * per_row;
+  for (size_t idx = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; idx < total;
+       idx += static_cast<size_t>(gridDim.x) * blockDim.x) {
+    const size_t t = idx / per_row;
+    const int c = static_cast<int>(idx - t * per_row) * kStep;
+    if constexpr (kVector) {
+      float v[8];
+      load8(in + t * in_stride + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float positive = fmaxf(v[i], 0.0f);
+        v[i] = positive * positive;
+      }
+      store8(out + t * out_stride + c, v);
+    } else {
+      const float positive = fmaxf(to_float(in[t * in_stride + c]), 0.0f);
+      out[t * out_stride + c] = from_float<T>(positive * positive);
     }
   }
 }
@@ -496,7 +532,7 @@ int rl_embedding_sum(int dtype, void* out, float* stream_out, const void* table,
 // x and out are `dtype`; residual and weight are float32.
 int rl_add_rmsnorm(int dtype, const void* x, float* residual, const float* weight, void* out,
                    const int* row_index, int rows, int hidden, float eps, int mode,
-                   int write_residual, const void* extra_rows, const float* extra_vector, int pdl,
+                   int write_residual, float x_scale, const void* extra_rows, const float* extra_vector, int pdl,
                    cudaStream_t stream) {
   if (rows == 0) return 0;
   if (mode < 0 || mode > 5 || ((mode == 1 || mode >= 3) && residual == nullptr) ||
@@ -511,7 +547,7 @@ int rl_add_rmsnorm(int dtype, const void* x, float* residual, const float* weigh
       const int threads = (hidden / 8 + 31) / 32 * 32;
       return rl::launch_kernel(rl::add_rmsnorm_kernel<scalar_t, scalar_t, true>, dim3(rows), dim3(threads), 0,
                                stream, pdl != 0, static_cast<const scalar_t*>(x), residual, weight,
-                               static_cast<scalar_t*>(out), row_index, hidden, eps, mode, write_residual,
+                               static_cast<scalar_t*>(out), row_index, hidden, eps, mode, write_residual, x_scale,
                                static_cast<const scalar_t*>(extra_rows), extra_vector);
     }
     const size_t smem = static_cast<size_t>(hidden) * sizeof(float);
@@ -526,7 +562,7 @@ int rl_add_rmsnorm(int dtype, const void* x, float* residual, const float* weigh
     }
     return rl::launch_kernel(kernel, dim3(rows), dim3(threads), smem, stream, pdl != 0,
                              static_cast<const scalar_t*>(x), residual, weight, static_cast<scalar_t*>(out),
-                             row_index, hidden, eps, mode, write_residual,
+                             row_index, hidden, eps, mode, write_residual, x_scale,
                              static_cast<const scalar_t*>(extra_rows), extra_vector);
   });
   return 0;
@@ -565,11 +601,13 @@ int rl_layernorm(int dtype, const void* x, float* residual, const float* weight,
   return 0;
 }
 
-int rl_sigmoid_gate(int dtype, const void* rows, const void* gate, int gate_stride, void* out, int tokens, int width,
-                    int pdl, cudaStream_t stream) {
+int rl_sigmoid_gate(int dtype, const void* rows, const void* gate, int gate_stride, void* out, int out_stride, int tokens,
+                    int width, int per, int pdl, cudaStream_t stream) {
   if (tokens == 0 || width == 0) return 0;
-  if (width < 0 || gate_stride < width) return static_cast<int>(cudaErrorInvalidValue);
-  const bool vector = width % 8 == 0 && gate_stride % 8 == 0 && rl::aligned16(rows) && rl::aligned16(gate) && rl::aligned16(out);
+  if (width < 0 || per < 1 || width % per != 0 || gate_stride < width / per || out_stride < width)
+    return static_cast<int>(cudaErrorInvalidValue);
+  const bool vector = width % 8 == 0 && out_stride % 8 == 0 && rl::aligned16(rows) && rl::aligned16(out) &&
+                      (per > 1 ? per % 8 == 0 : gate_stride % 8 == 0 && rl::aligned16(gate));
   const size_t total = static_cast<size_t>(tokens) * (vector ? width / 8 : width);
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
@@ -577,7 +615,23 @@ int rl_sigmoid_gate(int dtype, const void* rows, const void* gate, int gate_stri
     auto kernel = vector ? rl::sigmoid_gate_kernel<scalar_t, true> : rl::sigmoid_gate_kernel<scalar_t, false>;
     return rl::launch_kernel(kernel, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream, pdl != 0,
                              static_cast<const scalar_t*>(rows), static_cast<const scalar_t*>(gate), gate_stride,
-                             static_cast<scalar_t*>(out), tokens, width);
+                             static_cast<scalar_t*>(out), out_stride, tokens, width, per);
+  });
+  return 0;
+}
+
+int rl_relu_squared(int dtype, const void* in, int in_stride, void* out, int out_stride, int tokens, int width, int pdl,
+                    cudaStream_t stream) {
+  if (tokens == 0 || width == 0) return 0;
+  if (width < 0 || in_stride < width || out_stride < width) return static_cast<int>(cudaErrorInvalidValue);
+  const bool vector = width % 8 == 0 && in_stride % 8 == 0 && out_stride % 8 == 0 && rl::aligned16(in) && rl::aligned16(out);
+  const size_t total = static_cast<size_t>(tokens) * (vector ? width / 8 : width);
+  size_t blocks = (total + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  RL_DISPATCH_DTYPE(dtype, {
+    auto kernel = vector ? rl::relu_squared_kernel<scalar_t, true> : rl::relu_squared_kernel<scalar_t, false>;
+    return rl::launch_kernel(kernel, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream, pdl != 0,
+                             static_cast<const scalar_t*>(in), in_stride, static_cast<scalar_t*>(out), out_stride, tokens, width);
   });
   return 0;
 }

@@ -75,7 +75,16 @@ struct GemmArgs {
   // the gated unit of a fused gate/up product: glu_limit == 0: silu(gate) * up; glu_limit > 0: the clamped unit
   // g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(glu_alpha * g) * (u + 1)
   float glu_limit, glu_alpha;
+  // plain products: columns below this take the square of relu (a stacked product whose first rows are a
+  // feed-forward's); a multiple of 4
+  int relu2_columns;
+  float residual_scale;    // what the result is multiplied by when it joins the residual
 };
+
+__device__ __forceinline__ float relu_squared(float v) {
+  const float positive = fmaxf(v, 0.0f);
+  return positive * positive;
+}
 
 __device__ __forceinline__ float silu_mul(float gate, float up) {
   return __fdividef(gate, 1.0f + __expf(-gate)) * up;   // the result is rounded to bfloat16
@@ -338,6 +347,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gated_unit(v[j], (scaled ? u[j] * row_scale[c + j] : u[j]) + bias_up, args.glu_limit, args.glu_alpha);
           }
+          if (!kSwiglu && n < args.relu2_columns) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = relu_squared(v[j]);
+          }
           if (!kSwiglu && args.residual != nullptr) {
             const float norm_w = n < args.N ? args.norm_weight[n] : 0.0f;
 #pragma unroll
@@ -345,7 +358,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
               const int t = t0 + c + j;                 // the same for the whole warp
               if (t < args.T) {
                 const size_t at = static_cast<size_t>(t) * args.N + n;
-                const float sq = warp_sum(n < args.N ? store_for_norm(args, at, norm_w, args.residual[at] + v[j]) : 0.0f);
+                const float sq = warp_sum(n < args.N ? store_for_norm(args, at, norm_w, fmaf(args.residual_scale, v[j], args.residual[at])) : 0.0f);
                 if (lane == 0) args.sumsq_out[static_cast<size_t>(t) * (4 * args.n_tiles) + 4 * n_tile + quarter] = sq;
               }
             }
@@ -429,6 +442,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
         for (int r = 0; r < 4; ++r) {
           const float g = gate[r] * scale + bias_gate[r], u = up[r] * scale + bias_up[r];
           result[r] = kSwiglu ? gated_unit(g, u, args.glu_limit, args.glu_alpha) : g;
+          if (!kSwiglu && n + r < args.relu2_columns) result[r] = relu_squared(result[r]);
         }
         if (norm_follows) {
           float before[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -442,7 +456,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
           }
 #pragma unroll
           for (int r = 0; r < 4; ++r) {
-            before[r] += result[r];                                // the new residual
+            before[r] = fmaf(args.residual_scale, result[r], before[r]);     // the new residual
             result[r] = before[r] * norm_w[r];
             if (n + r < args.N) squares += before[r] * before[r];
           }
@@ -576,11 +590,18 @@ extern "C" {
 // multiplied by rsqrt(sum(sumsq_in[t]) / norm_size + norm_eps).
 // `bias` (float32 [n_out], SwiGLU [2 n_out]; may be null) is added to every row after that scale.
 // `glu_limit` > 0 (only with swiglu): the gated unit is the clamped one, see GemmArgs.
+// `x_pitch`: elements from a row of x to the next (0 = k; a multiple of 8), for an x that is some columns of wider rows.
+// `relu2_columns` (a plain product without a norm behind it): the first so many columns of the result, after the bias,
+// become max(v, 0)^2.  `residual_scale` multiplies the result where it joins the residual.
 int rl_gemm_bf16_norm(const void* x, const void* w, void* out, int tokens, int n_out, int k, int swiglu, int pdl,
                       int k_split, float* residual, const float* norm_weight, float* sumsq_out,
                       const float* sumsq_in, int sumsq_count, float norm_eps, int norm_size, const float* bias,
-                      float glu_limit, float glu_alpha, int* fault, cudaStream_t stream) {
+                      float glu_limit, float glu_alpha, int x_pitch, int relu2_columns, float residual_scale, int* fault,
+                      cudaStream_t stream) {
   if (tokens == 0 || n_out == 0) return 0;
+  if (x_pitch != 0 && (x_pitch < k || x_pitch % 8 != 0)) return static_cast<int>(cudaErrorInvalidValue);
+  if (relu2_columns < 0 || relu2_columns > n_out || (relu2_columns > 0 && (swiglu != 0 || residual != nullptr)))
+    return static_cast<int>(cudaErrorInvalidValue);
   if (glu_limit < 0.0f || (glu_limit > 0.0f && swiglu == 0)) return static_cast<int>(cudaErrorInvalidValue);
   if (tokens < 0 || n_out < 0 || k <= 0 || k % 8 != 0 || k_split < 0 || k_split > 8 ||
       (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
@@ -612,7 +633,7 @@ int rl_gemm_bf16_norm(const void* x, const void* w, void* out, int tokens, int n
   CUtensorMap map_w, map_x;
   int status = rl::make_map(&map_w, w, static_cast<long long>(n_out) * (swiglu ? 2 : 1), k, tile_rows);
   if (status != 0) return status;
-  status = rl::make_map(&map_x, x, tokens, k, bn);
+  status = rl::make_map(&map_x, x, tokens, k, bn, x_pitch);
   if (status != 0) return status;
   rl::GemmArgs args;
   args.out = static_cast<rl::bf16*>(out);
@@ -634,6 +655,7 @@ int rl_gemm_bf16_norm(const void* x, const void* w, void* out, int tokens, int n
   args.inv_norm_size = norm_size > 0 ? 1.0f / static_cast<float>(norm_size) : 0.0f;
   args.bias = bias;
   args.glu_limit = glu_limit; args.glu_alpha = glu_alpha;
+  args.relu2_columns = relu2_columns; args.residual_scale = residual_scale;
 #define RL_GEMM_CASE(SW, BNV) \
   if ((swiglu != 0) == SW && bn == BNV) return rl::launch_gemm<SW, BNV>(map_w, map_x, args, k_split, stream);
   RL_GEMM_CASE(false, 16) RL_GEMM_CASE(false, 32) RL_GEMM_CASE(false, 64) RL_GEMM_CASE(false, 128)
@@ -646,7 +668,7 @@ int rl_gemm_bf16_norm(const void* x, const void* w, void* out, int tokens, int n
 int rl_gemm_bf16(const void* x, const void* w, void* out, int tokens, int n_out, int k, int swiglu, int pdl,
                  int k_split, int* fault, cudaStream_t stream) {
   return rl_gemm_bf16_norm(x, w, out, tokens, n_out, k, swiglu, pdl, k_split, nullptr, nullptr, nullptr, nullptr, 0,
-                           0.0f, 0, nullptr, 0.0f, 0.0f, fault, stream);
+                           0.0f, 0, nullptr, 0.0f, 0.0f, 0, 0, 1.0f, fault, stream);
 }
 
 // columns of the table of partial sums of squares that a product of `n_out` output columns writes per token

@@ -492,7 +492,9 @@ __global__ void rope_unit_write_kernel(const RopeUnitArgs a) {
 // whole query row (hq * d numbers, heads laid out in d with their padding at zero), q <- q * rsqrt(sum(q^2) /
 // q_count + eps) * q_weight, q_count the true number of entries and q_weight one float per laid-out entry; the same
 // for k.  Then the first `rotary` entries of every q and k head rotate by halves (entry i with i + rotary / 2, angle
-// position * inv_freq[i], sine and cosine formed here in float32), q goes to q_out and k, v into the pages.
+// position * inv_freq[i], sine and cosine formed here in float32), or in neighbouring pairs (`neighbours`: entry 2i with
+// 2i + 1); q goes to q_out and k, v into the pages.  `values_are_keys`: the row has no v columns, the values are the k
+// columns as they come (neither normed nor rotated).
 // One block per token; the sums run down the block's fixed tree, so a token's result does not depend on the step.
 // All arithmetic float32, one rounding at the store.  kv_dest null: the row holds queries only.  Columns of the row
 // behind the heads (a gate's, brought along by the same product) are not read.
@@ -518,7 +520,7 @@ __global__ void row_norm_rope_write_vec_kernel(const T* __restrict__ qkv, int ro
                                                const int* __restrict__ positions, const int* __restrict__ kv_dest,
                                                T* __restrict__ q_out, T* __restrict__ cache, int hq, int hkv, int d,
                                                int rotary, int q_count, int k_count, float eps, int page_size,
-                                               int num_pages, int* __restrict__ fault) {
+                                               int num_pages, int neighbours, int values_are_keys, int* __restrict__ fault) {
   extern __shared__ __align__(16) float row_f32[];      // [hq * d] q, then [hkv * d] k
   __shared__ float scratch[32];
   __shared__ float cs[kMaxHeadDim / 2], sn[kMaxHeadDim / 2];
@@ -539,7 +541,7 @@ __global__ void row_norm_rope_write_vec_kernel(const T* __restrict__ qkv, int ro
   }
   pdl_wait();
   float sum_q = 0.0f, sum_k = 0.0f;
-  const int chunks = (q_width + 2 * k_width) >> 3;
+  const int chunks = (q_width + (values_are_keys ? 1 : 2) * k_width) >> 3;
   for (int c = threadIdx.x; c < chunks; c += blockDim.x) {
     const int at = c << 3;
     float v[8];
@@ -550,8 +552,9 @@ __global__ void row_norm_rope_write_vec_kernel(const T* __restrict__ qkv, int ro
 #pragma unroll
       for (int e = 0; e < 8; ++e) sq += v[e] * v[e];
       if (at < q_width) sum_q += sq; else sum_k += sq;
-    } else if (!bad_page) {
-      const int idx = at - q_width - k_width, head = idx / d, i = idx - head * d;
+    }
+    if (at >= q_width + (values_are_keys ? 0 : k_width) && !bad_page) {
+      const int idx = at - q_width - (values_are_keys ? 0 : k_width), head = idx / d, i = idx - head * d;
       store8_as(cache + (((static_cast<size_t>(page) * 2 + 1) * hkv + head) * page_size + offset) * d + i, v);
     }
   }
@@ -571,15 +574,28 @@ __global__ void row_norm_rope_write_vec_kernel(const T* __restrict__ qkv, int ro
     const int head = idx / d, i0 = idx - head * d;
     float wv[8], v[8];
     load8(w + idx, wv);
+    if (neighbours) {      // a pair lies in one thread's eight
+      load8(src + idx, v);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      const int i = i0 + e;
-      v[e] = src[idx + e] * inv * wv[e];
-      if (i < rotary) {
-        const int other_at = i < half ? idx + e + half : idx + e - half;
-        const float other = src[other_at] * inv * w[other_at];
-        const int pair = i < half ? i : i - half;
-        v[e] = i < half ? v[e] * cs[pair] - other * sn[pair] : v[e] * cs[pair] + other * sn[pair];
+      for (int e = 0; e < 8; e += 2) {
+        const float a = v[e] * inv * wv[e], b = v[e + 1] * inv * wv[e + 1];
+        const int i = i0 + e;
+        const bool turns = i < rotary;
+        const float co = turns ? cs[i >> 1] : 1.0f, si = turns ? sn[i >> 1] : 0.0f;
+        v[e] = turns ? a * co - b * si : a;
+        v[e + 1] = turns ? b * co + a * si : b;
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int i = i0 + e;
+        v[e] = src[idx + e] * inv * wv[e];
+        if (i < rotary) {
+          const int other_at = i < half ? idx + e + half : idx + e - half;
+          const float other = src[other_at] * inv * w[other_at];
+          const int pair = i < half ? i : i - half;
+          v[e] = i < half ? v[e] * cs[pair] - other * sn[pair] : v[e] * cs[pair] + other * sn[pair];
+        }
       }
     }
     if (is_q) {
@@ -596,12 +612,12 @@ extern "C" int rl_row_norm_rope_write(int dtype, const void* qkv, int row_width,
                                       const float* k_weight, const float* inv_freq, const int* positions,
                                       const int* kv_dest, void* q_out, void* cache, int tokens, int hq, int hkv, int d,
                                       int rotary, int q_count, int k_count, float eps, int page_size, int num_pages,
-                                      int* fault, int pdl, cudaStream_t stream) {
+                                      int neighbours, int values_are_keys, int* fault, int pdl, cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (d <= 0 || d > rl::kMaxHeadDim || rotary < 0 || rotary > d || (rotary & 1) || hq <= 0 || q_count < 1 ||
       q_weight == nullptr || (rotary > 0 && inv_freq == nullptr) ||
       (kv_dest != nullptr && (hkv <= 0 || k_count < 1 || k_weight == nullptr || cache == nullptr || page_size <= 0)) ||
-      row_width < (kv_dest ? (hq + 2 * hkv) * d : hq * d))
+      row_width < (kv_dest ? (hq + (values_are_keys ? 1 : 2) * hkv) * d : hq * d))
     return static_cast<int>(cudaErrorInvalidValue);
   const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const int staged = (hq + (kv_dest ? hkv : 0)) * d;
@@ -619,7 +635,7 @@ extern "C" int rl_row_norm_rope_write(int dtype, const void* qkv, int row_width,
       return rl::launch_kernel(kernel, dim3(tokens), dim3(threads), smem, stream, pdl != 0,
                                static_cast<const scalar_t*>(qkv), row_width, q_weight, k_weight, inv_freq, positions,
                                kv_dest, static_cast<scalar_t*>(q_out), static_cast<scalar_t*>(cache), hq, hkv, d, rotary,
-                               q_count, k_count, eps, page_size, num_pages, fault);
+                               q_count, k_count, eps, page_size, num_pages, neighbours, values_are_keys, fault);
     });
   }
   return static_cast<int>(cudaErrorInvalidValue);      // sizes or addresses that are no multiples of 16 bytes

@@ -299,11 +299,12 @@ static EncodeTiled encode_tiled() {
 
 
 // A [rows, cols] row-major bf16 matrix read in boxes of box_rows x 64 with the 128-byte swizzle.
-static int make_map(CUtensorMap* map, const void* base, long long rows, long long cols, int box_rows) {
+// `pitch`: elements from a row to the next (a multiple of 8; 0 = cols), for rows that are some columns of wider ones.
+static int make_map(CUtensorMap* map, const void* base, long long rows, long long cols, int box_rows, long long pitch = 0) {
   EncodeTiled encode = encode_tiled();
   if (encode == nullptr) return static_cast<int>(cudaErrorNotSupported);
   const cuuint64_t dims[2] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(rows)};
-  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(cols) * 2};
+  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(pitch > 0 ? pitch : cols) * 2};
   const cuuint32_t box[2] = {64u, static_cast<cuuint32_t>(box_rows)};
   const cuuint32_t elem[2] = {1, 1};
   const CUresult r = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides,

@@ -25,7 +25,7 @@ class GroupView:
         kv_dest: int32 ``[T]``; ``page * page_size + offset`` where each token of the step
             writes its key and value.
         page_size: Tokens per page.
-        window: Positions a query reaches back (its own included); 0 = all of them.
+        window: Most positions a query sees, its own included (a window, a chunk); 0 = all of them.
     """
 
     block_table: torch.Tensor

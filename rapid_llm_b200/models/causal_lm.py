@@ -132,6 +132,8 @@ class CausalLM:
             x = embedded = self.embedding.forward(batch, *own)
             residual = None
         schedule = self.spec.schedule
+        if residual is not None and self.layers[schedule[0].layer].takes_open_stream:
+            x = None                  # the stream is complete: the first layer has nothing to add to it
         for position, entry in enumerate(schedule):
             # the norm that the next layer starts with may ride on this layer's last product, unless
             # something joins the stream in between

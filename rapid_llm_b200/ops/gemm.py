@@ -67,7 +67,8 @@ kernels.BEFORE_LAUNCH = flush
 def _product(x, weight, out, fault, defer: bool, **options) -> None:
     """One tensor-core product: queued if the caller allows it, else run at once (after the queue)."""
     options = {name: value for name, value in options.items() if value is not None and value is not False}
-    if defer and CHAIN and x.shape[0] <= kernels.GEMM_CHAIN_MAX_TOKENS:
+    chains = "relu2_columns" not in options and "residual_scale" not in options and x.is_contiguous()
+    if defer and CHAIN and chains and x.shape[0] <= kernels.GEMM_CHAIN_MAX_TOKENS:
         if _PENDING and (len(_PENDING) == kernels.GEMM_CHAIN_MAX_PHASES or _PENDING[0]["x"].shape[0] != x.shape[0]
                          or _PENDING_FAULT[0] is not fault):
             flush()
@@ -80,7 +81,7 @@ def _product(x, weight, out, fault, defer: bool, **options) -> None:
 
 @dataclass
 class FollowingNorm:
-    """A norm ``y = r * rsqrt(mean(r^2) + eps) * weight`` of ``r = residual + (a product's result)``,
+    """A norm ``y = r * rsqrt(mean(r^2) + eps) * weight`` of ``r = residual + scale * (a product's result)``,
     offered to that product: ``residual`` (float32, updated in place) and the norm's float32 ``weight``;
     ``workspace`` lends the buffers of the result."""
 
@@ -88,6 +89,7 @@ class FollowingNorm:
     weight: torch.Tensor
     eps: float
     workspace: Any
+    scale: float = 1.0        # what the product's result is multiplied by where it joins the residual
 
 
 @dataclass
@@ -136,8 +138,11 @@ def _bias_as(bias: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 
 
 def linear(x, weight: torch.Tensor, out: torch.Tensor, fault: torch.Tensor | None = None, *,
-           then_norm: FollowingNorm | None = None, bias: torch.Tensor | None = None, defer: bool = False):
-    """``out[T, N] = x[T, K] @ weight[N, K]^T (+ bias[N], float32)``; all on the GPU, same dtype.
+           then_norm: FollowingNorm | None = None, bias: torch.Tensor | None = None, defer: bool = False,
+           relu2_columns: int = 0):
+    """``out[T, N] = x[T, K] @ weight[N, K]^T (+ bias[N], float32)``; all on the GPU, same dtype.  ``x`` may be a view of
+    some columns of wider rows.  The first ``relu2_columns`` columns become ``max(v, 0)^2``: in the tensor-core product's
+    epilogue, by a kernel behind the library's and the 32-bit product.
 
     ``x`` may be :class:`ScaledRows`.  With ``then_norm`` the product may take the norm along:
     it then returns :class:`ScaledRows` (the residual is updated, ``out`` is not written);
@@ -149,10 +154,13 @@ def linear(x, weight: torch.Tensor, out: torch.Tensor, fault: torch.Tensor | Non
         raise kernels.KernelError("linear: tensors must live on a CUDA device; there is no CPU path")
     if x.dtype != weight.dtype or out.dtype != x.dtype:
         raise kernels.KernelError(f"linear: dtypes differ ({x.dtype}, {weight.dtype}, {out.dtype})")
-    if x.dtype == torch.float32:
-        return kernels.gemm_f32(x, weight, out, bias)
+    if relu2_columns and then_norm is not None:
+        raise kernels.KernelError("linear: a norm does not ride on a product whose columns pass an activation")
     if x.shape[0] == 0:
         return out
+    if x.dtype == torch.float32:
+        kernels.gemm_f32(x, weight, out, bias)
+        return _square_columns(out, relu2_columns)
     if fault is not None and use_tensor_core_kernel(x, weight):
         rows, width = out.shape
         if (then_norm is not None and FUSE_NORMS and rows <= kernels.GEMM_NORM_MAX_TOKENS and width % 8 == 0
@@ -160,20 +168,26 @@ def linear(x, weight: torch.Tensor, out: torch.Tensor, fault: torch.Tensor | Non
             normed = then_norm.workspace.get("normed", rows, width, x.dtype)
             sumsq = then_norm.workspace.get("normed_sumsq", rows, kernels.gemm_bf16_sumsq_count(width), torch.float32)
             _product(x, weight, normed, fault, defer, residual=then_norm.residual, norm_weight=then_norm.weight,
-                     sumsq_out=sumsq, bias=bias, **scale)
+                     sumsq_out=sumsq, bias=bias, residual_scale=then_norm.scale if then_norm.scale != 1.0 else None, **scale)
             return ScaledRows(normed, sumsq, then_norm.eps, width)
-        _product(x, weight, out, fault, defer, bias=bias, **scale)
+        _product(x, weight, out, fault, defer, bias=bias, relu2_columns=relu2_columns or None, **scale)
         return out
     flush()
     if scale:
         raise kernels.KernelError("linear: rows with an open scale need the tensor-core product")
     if (FORCE == "pair" and fault is not None and kernels.gemm_bf16_supports(x, weight)
-            and kernels.gemm_bf16_pair_takes(x.shape[0], out.shape[1], False)):
-        return kernels.gemm_bf16_pair(x, weight, out, fault, bias=bias)
+            and x.is_contiguous() and kernels.gemm_bf16_pair_takes(x.shape[0], out.shape[1], False)):
+        return _square_columns(kernels.gemm_bf16_pair(x, weight, out, fault, bias=bias), relu2_columns)
     if bias is None:
         torch.mm(x, weight.t(), out=out)
     else:
         torch.addmm(_bias_as(bias, x.dtype), x, weight.t(), out=out)
+    return _square_columns(out, relu2_columns)
+
+
+def _square_columns(out: torch.Tensor, columns: int) -> torch.Tensor:
+    if columns:
+        kernels.relu_squared(out[:, :columns], out[:, :columns])
     return out
 
 

@@ -117,14 +117,15 @@ def core() -> ctypes.CDLL:
     lib = load_library("core")
     if not _SIGNATURES_SET:
         lib.rl_embedding.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p]
-        lib.rl_add_rmsnorm.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
+        lib.rl_add_rmsnorm.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p]
         lib.rl_layernorm.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                      c_float, c_float, c_int, c_float, c_int, c_void_p]
         lib.rl_row_norm_rope_write.argtypes = [
             c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p,
+            c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
         ]
-        lib.rl_sigmoid_gate.argtypes = [c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]
+        lib.rl_sigmoid_gate.argtypes = [c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
+        lib.rl_relu_squared.argtypes = [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.rl_silu_mul.argtypes = [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
         lib.rl_clamped_glu.argtypes = [c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p]
         lib.rl_rope_unit_write.argtypes = [
@@ -140,7 +141,7 @@ def core() -> ctypes.CDLL:
         ]
         lib.rl_attention_generic.argtypes = [
             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p,
+            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p,
         ]
         lib.rl_embedding_sum.argtypes = [
             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
@@ -153,7 +154,7 @@ def core() -> ctypes.CDLL:
         ]
         for name in (
             "rl_embedding", "rl_embedding_sum", "rl_scatter_rows", "rl_add_rmsnorm", "rl_silu_mul", "rl_to_float", "rl_clamped_glu",
-            "rl_rope_unit_write", "rl_layernorm", "rl_row_norm_rope_write", "rl_sigmoid_gate",
+            "rl_rope_unit_write", "rl_layernorm", "rl_row_norm_rope_write", "rl_sigmoid_gate", "rl_relu_squared",
             "rl_qk_norm_rope_write", "rl_attention_generic", "rl_gemm_f32", "rl_sample",
         ):
             getattr(lib, name).restype = c_int
@@ -239,8 +240,9 @@ def add_rmsnorm(
     row_index: torch.Tensor | None = None,
     extra_rows: torch.Tensor | None = None,
     extra_vector: torch.Tensor | None = None,
+    x_scale: float = 1.0,
 ) -> torch.Tensor:
-    """RMSNorm of ``x`` (mode 0 or 2) or of ``x + residual`` (mode 1), float32 math.
+    """RMSNorm of ``x`` (mode 0 or 2) or of ``x_scale * x + residual`` (mode 1), float32 math.
 
     ``residual`` is the float32 residual stream ``[T, H]``; with ``write_residual`` the
     sum is stored back into it.  ``row_index`` (int32) selects the input rows; ``out`` then
@@ -265,7 +267,7 @@ def add_rmsnorm(
         raise KernelError("add_rmsnorm: residual must have the shape of x")
     _check(
         core().rl_add_rmsnorm(dtype_tag(x.dtype), _ptr(x), _ptr(residual), _ptr(weight), _ptr(out),
-                              _ptr(row_index), rows, hidden, float(eps), mode, int(write_residual),
+                              _ptr(row_index), rows, hidden, float(eps), mode, int(write_residual), float(x_scale),
                               _ptr(extra_rows), _ptr(extra_vector), int(PDL), _stream()),
         f"add_rmsnorm(hidden={hidden})",
     )
@@ -283,7 +285,7 @@ def stream_rmsnorm(residual: torch.Tensor, weight: torch.Tensor, out: torch.Tens
     if weight.numel() != hidden or out.shape != (rows, hidden):
         raise KernelError("stream_rmsnorm: shapes of residual, weight and out do not agree")
     _check(core().rl_add_rmsnorm(dtype_tag(out.dtype), None, _ptr(residual), _ptr(weight), _ptr(out), _ptr(row_index),
-                                 rows, hidden, float(eps), 3, 0, None, None, int(PDL), _stream()), "stream_rmsnorm")
+                                 rows, hidden, float(eps), 3, 0, 1.0, None, None, int(PDL), _stream()), "stream_rmsnorm")
     return out
 
 
@@ -296,7 +298,7 @@ def join_rmsnorm(x: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, 
     if residual.shape != x.shape or out.shape != x.shape or out.dtype != x.dtype or weight.numel() != x.shape[-1]:
         raise KernelError("join_rmsnorm: shapes of x, residual, weight and out do not agree")
     _check(core().rl_add_rmsnorm(dtype_tag(x.dtype), _ptr(x), _ptr(residual), _ptr(weight), _ptr(out), None,
-                                 x.shape[0], x.shape[1], float(eps), 4, 1, None, None, int(PDL), _stream()), "join_rmsnorm")
+                                 x.shape[0], x.shape[1], float(eps), 4, 1, 1.0, None, None, int(PDL), _stream()), "join_rmsnorm")
     return out
 
 
@@ -335,18 +337,20 @@ def row_norm_rope_write(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: in
                         q_weight: torch.Tensor, k_weight: torch.Tensor | None, q_count: int, k_count: int,
                         inv_freq: torch.Tensor | None, positions: torch.Tensor, eps: float, fault: torch.Tensor,
                         kv_dest: torch.Tensor | None = None, cache: torch.Tensor | None = None,
-                        page_size: int = 1) -> torch.Tensor:
+                        page_size: int = 1, neighbours: bool = False, values_are_keys: bool = False) -> torch.Tensor:
     """RMS norm of q over ALL its heads at once (and of k likewise), ``q * rsqrt(sum(q^2) / q_count + eps) * q_weight``
     with one weight per laid-out entry, then rotation by halves of the first ``2 len(inv_freq)`` entries of every q and
-    k head (angles ``position * inv_freq`` formed in float32), q to ``q_out``, k and v into the pages.  ``qkv`` is
-    ``[T, (Hq + 2 Hkv) D]``, or ``[T, Hq D]`` with ``kv_dest`` ``None`` (queries only)."""
+    k head (angles ``position * inv_freq`` formed in float32; ``neighbours``: entries ``2i`` and ``2i + 1`` turn
+    together instead of ``i`` and ``i + len(inv_freq)``), q to ``q_out``, k and v into the pages.  ``qkv`` is
+    ``[T, (Hq + 2 Hkv) D]``, or ``[T, Hq D]`` with ``kv_dest`` ``None`` (queries only), or ``[T, (Hq + Hkv) D]`` with
+    ``values_are_keys``: the values are the k columns as they come.  It may be a view of some columns of wider rows."""
     _need_cuda(qkv, q_out, q_weight, k_weight, inv_freq, positions, fault, kv_dest, cache)
-    _contig("qkv", qkv), _contig("q_out", q_out), _contig("cache", cache), _contig("inv_freq", inv_freq)
+    _contig("q_out", q_out), _contig("cache", cache), _contig("inv_freq", inv_freq)
     for name, tensor in (("q_weight", q_weight), ("k_weight", k_weight), ("inv_freq", inv_freq)):
         _expect(name, tensor, torch.float32), _contig(name, tensor)
     _expect("positions", positions, torch.int32), _expect("kv_dest", kv_dest, torch.int32)
     tokens, row_width = qkv.shape
-    heads_in = num_heads + 2 * num_kv_heads if kv_dest is not None else num_heads
+    heads_in = num_heads + (1 if values_are_keys else 2) * num_kv_heads if kv_dest is not None else num_heads
     if row_width < heads_in * head_dim or q_out.numel() != tokens * num_heads * head_dim or q_out.dtype != qkv.dtype:
         raise KernelError("row_norm_rope_write: qkv or q_out do not fit the heads")      # columns behind the heads are not read
     if q_weight.numel() != num_heads * head_dim or (kv_dest is not None and (k_weight is None or k_weight.numel() != num_kv_heads * head_dim)):
@@ -358,22 +362,34 @@ def row_norm_rope_write(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: in
         num_pages = cache.shape[0]
     rotary = 0 if inv_freq is None else 2 * inv_freq.numel()
     _check(core().rl_row_norm_rope_write(
-        dtype_tag(qkv.dtype), _ptr(qkv), row_width, _ptr(q_weight), _ptr(k_weight), _ptr(inv_freq), _ptr(positions),
+        dtype_tag(qkv.dtype), _ptr(qkv), _row_stride("qkv", qkv), _ptr(q_weight), _ptr(k_weight), _ptr(inv_freq), _ptr(positions),
         _ptr(kv_dest), _ptr(q_out), _ptr(cache), tokens, num_heads, num_kv_heads, head_dim, rotary, int(q_count),
-        int(k_count), float(eps), page_size, num_pages, _ptr(fault), int(PDL), _stream()),
+        int(k_count), float(eps), page_size, num_pages, int(neighbours), int(values_are_keys), _ptr(fault), int(PDL), _stream()),
         f"row_norm_rope_write(head_dim={head_dim})")
     return q_out
 
 
 def sigmoid_gate(rows: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """``out = rows * sigmoid(gate)`` entry by entry (float32 arithmetic); ``gate`` may be a view of some columns of
-    wider rows."""
+    """``out = rows * sigmoid(gate)`` (float32 arithmetic): entry by entry, or, with a ``gate [T, heads]``, one number
+    for all entries of a head.  ``gate`` and ``out`` may be views of some columns of wider rows."""
     _need_cuda(rows, gate, out)
-    _contig("rows", rows), _contig("out", out)
-    if gate.shape != rows.shape or out.shape != rows.shape or gate.dtype != rows.dtype or out.dtype != rows.dtype:
+    _contig("rows", rows)
+    if (gate.shape[0] != rows.shape[0] or rows.shape[1] % gate.shape[1] or out.shape != rows.shape
+            or gate.dtype != rows.dtype or out.dtype != rows.dtype):
         raise KernelError("sigmoid_gate: shapes or dtypes do not agree")
     _check(core().rl_sigmoid_gate(dtype_tag(rows.dtype), _ptr(rows), _ptr(gate), _row_stride("gate", gate), _ptr(out),
-                                  rows.shape[0], rows.shape[1], int(PDL), _stream()), "sigmoid_gate")
+                                  _row_stride("out", out), rows.shape[0], rows.shape[1], rows.shape[1] // gate.shape[1],
+                                  int(PDL), _stream()), "sigmoid_gate")
+    return out
+
+
+def relu_squared(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out = max(x, 0)^2`` (float32 arithmetic); both may be views of some columns of wider rows, and the same one."""
+    _need_cuda(x, out)
+    if out.shape != x.shape or out.dtype != x.dtype:
+        raise KernelError("relu_squared: shapes or dtypes do not agree")
+    _check(core().rl_relu_squared(dtype_tag(x.dtype), _ptr(x), _row_stride("x", x), _ptr(out), _row_stride("out", out),
+                                  x.shape[0], x.shape[1], int(PDL), _stream()), "relu_squared")
     return out
 
 
@@ -515,8 +531,10 @@ def attention_generic(
     fault: torch.Tensor,
     softcap: float = 0.0,
     sink: torch.Tensor | None = None,
+    chunk: int = 0,
 ) -> torch.Tensor:
-    """Causal attention of every token of the step over its request's cached keys.  ``softcap`` > 0 squashes the
+    """Causal attention of every token of the step over its request's cached keys: all of them, the last ``window``
+    positions, or (``chunk`` > 0) those of the position's own chunk, counted from position 0.  ``softcap`` > 0 squashes the
     scaled scores to ``softcap * tanh(s / softcap)``; ``sink`` (float32 ``[heads]``) adds ``exp(sink[h])`` to every
     row's denominator."""
     _need_cuda(q, cache, out, positions, token_slot, block_table, fault, sink)
@@ -539,7 +557,7 @@ def attention_generic(
         core().rl_attention_generic(
             dtype_tag(q.dtype), _ptr(q), _ptr(cache), _ptr(out), _ptr(positions), _ptr(token_slot),
             _ptr(block_table), tokens, num_heads, num_kv_heads, head_dim, cache.shape[3],
-            cache.shape[0], block_table.shape[1], block_table.shape[0], int(window), float(scale),
+            cache.shape[0], block_table.shape[1], block_table.shape[0], int(window), int(chunk), float(scale),
             float(softcap), _ptr(sink), int(cache.shape[1]), _ptr(fault), _stream(),
         ),
         f"attention_generic(head_dim={head_dim})",
@@ -554,6 +572,7 @@ CHUNK_TILE_ROWS_TC = 256   # ... of the tcgen05 kernel (head size 128, unsplit k
 DECODE_TILE_ROWS = 16      # ... of a decode tile
 TC_HEAD_DIM = 128
 DECODE_TC_KEYS = 128      # keys per block of the tcgen05 decode kernel
+MMA_KEYS = 64             # ... of the mma.sync tiles
 
 
 def attention_tc_takes(head_dim: int, page_size: int) -> bool:
@@ -571,7 +590,7 @@ def attention_lib(head_dim: int) -> ctypes.CDLL:
         lib.rl_attention_mma.argtypes = [
             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
+            c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
         ]
         lib.rl_attention_mma.restype = c_int
         lib.rl_attention_decode_max_clusters.argtypes = [c_int]
@@ -628,6 +647,7 @@ def attention_mma(
     decode_splits: int = 0,
     softcap: float = 0.0,
     sink: torch.Tensor | None = None,
+    chunk: int = 0,
 ) -> torch.Tensor:
     """bfloat16 paged causal attention over work items the host cut the step into.
 
@@ -646,8 +666,9 @@ def attention_mma(
     ``splits == 1``, where that kernel applies, up to 16.
 
     ``softcap`` > 0 squashes the scaled scores to ``softcap * tanh(s / softcap)``; ``sink`` (float32 ``[heads]``)
-    adds ``exp(sink[h])`` to every row's denominator, once.  The tcgen05 chunk tiles and the mma.sync tiles take
-    both; with either one the decode tiles run on mma.sync (and have no split count of their own).
+    adds ``exp(sink[h])`` to every row's denominator, once.  All tiles take a sink; with squashed scores the decode
+    tiles run on mma.sync (and have no split count of their own).  A position sees all keys up to its own, or the last
+    ``window`` of them, or (``chunk`` > 0) those of its own chunk, chunks being counted from position 0.
     """
     _need_cuda(q, cache, out, chunk_items, decode_items, part_out, part_lse, cu_seqlens, entry_start,
                entry_slot, block_table, fault, sink)
@@ -679,7 +700,7 @@ def attention_mma(
             _ptr(q), _ptr(cache), _ptr(out), _ptr(part_out), _ptr(part_lse), _ptr(chunk_items), n_chunk,
             _ptr(decode_items), n_decode, _ptr(cu_seqlens), _ptr(entry_start), _ptr(entry_slot),
             _ptr(block_table), tokens, num_heads, num_kv_heads, head_dim, cache.shape[3], cache.shape[0],
-            block_table.shape[1], block_table.shape[0], int(window), int(splits), float(scale),
+            block_table.shape[1], block_table.shape[0], int(window), int(chunk), int(splits), float(scale),
             _ptr(fault), int(PDL), {"auto": 0, "mma": 1, "deep": 2, "shallow": 3}[decode_kernel], int(decode_rows), int(chunk_rows),
             int(decode_splits), float(softcap), _ptr(sink), int(cache.shape[1]), _stream(),
         ),
@@ -719,7 +740,7 @@ def gemm_lib() -> ctypes.CDLL:
         lib.rl_gemm_bf16.restype = c_int
         lib.rl_gemm_bf16_norm.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, ctypes.c_float, c_int,
-                                          c_void_p, c_float, c_float, c_void_p, c_void_p]
+                                          c_void_p, c_float, c_float, c_int, c_int, c_float, c_void_p, c_void_p]
         lib.rl_gemm_bf16_norm.restype = c_int
         lib.rl_gemm_bf16_sumsq_count.argtypes = [c_int]
         lib.rl_gemm_bf16_sumsq_count.restype = c_int
@@ -729,7 +750,7 @@ def gemm_lib() -> ctypes.CDLL:
 
 def gemm_bf16_supports(x: torch.Tensor, w: torch.Tensor) -> bool:
     """Whether the tensor-core product takes these operands (TMA wants 16-byte rows)."""
-    return x.shape[1] % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
+    return x.shape[1] % 8 == 0 and (x.shape[0] <= 1 or x.stride(0) % 8 == 0) and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
 
 
 GEMM_NORM_MAX_TOKENS = 64   # most rows of a product that carries a norm's add or a norm's open scale
@@ -744,8 +765,10 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, fault: torch.
               k_split: int = 0, residual: torch.Tensor | None = None, norm_weight: torch.Tensor | None = None,
               sumsq_out: torch.Tensor | None = None, sumsq_in: torch.Tensor | None = None,
               norm_eps: float = 0.0, norm_size: int = 0, bias: torch.Tensor | None = None,
-              glu_limit: float = 0.0, glu_alpha: float = 1.0) -> torch.Tensor:
-    """``out[T, N] = x[T, K] @ w[N, K]^T`` in bfloat16 on the tcgen05 tensor cores.
+              glu_limit: float = 0.0, glu_alpha: float = 1.0, relu2_columns: int = 0,
+              residual_scale: float = 1.0) -> torch.Tensor:
+    """``out[T, N] = x[T, K] @ w[N, K]^T`` in bfloat16 on the tcgen05 tensor cores; ``x`` may be a view of some columns
+    of wider rows.  The first ``relu2_columns`` columns of a plain product become ``max(v, 0)^2`` (after the bias).
 
     With ``swiglu``, ``w`` is ``[2 N, K]`` (gate rows, then up rows) and
     ``out = silu(x @ gate^T) * (x @ up^T)`` without the ``[T, 2 N]`` intermediate; with ``glu_limit`` > 0 the unit
@@ -755,7 +778,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, fault: torch.
 
     A norm between two products rides on them (at most :data:`GEMM_NORM_MAX_TOKENS` rows).
     With ``residual`` (float32 ``[T, N]``), ``norm_weight`` (float32 ``[N]``) and ``sumsq_out``
-    (float32 ``[T, gemm_bf16_sumsq_count(N)]``) the product is added to ``residual`` in place,
+    (float32 ``[T, gemm_bf16_sumsq_count(N)]``) the product, times ``residual_scale``, is added to ``residual`` in place,
     ``out = residual * norm_weight`` and ``sumsq_out`` receives partial sums of the new
     residual's squares.  With ``sumsq_in`` (such a table), ``norm_eps`` and ``norm_size``, row
     ``t`` of the product is multiplied by ``rsqrt(sum(sumsq_in[t]) / norm_size + norm_eps)``
@@ -768,7 +791,9 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, fault: torch.
         if bias.shape != (w.shape[0],):
             raise KernelError(f"gemm_bf16: bias of shape {tuple(bias.shape)} for a weight of {w.shape[0]} rows")
     for name, tensor in (("x", x), ("w", w), ("out", out)):
-        _expect(name, tensor, torch.bfloat16), _contig(name, tensor)
+        _expect(name, tensor, torch.bfloat16)
+    x_pitch = _row_stride("x", x) if x.shape[0] > 1 else 0      # 0: as wide as x itself
+    _contig("w", w), _contig("out", out)
     tokens, k = x.shape
     n_out = out.shape[1]
     if w.shape != ((2 if swiglu else 1) * n_out, k) or out.shape[0] != tokens:
@@ -797,7 +822,8 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, fault: torch.
             _ptr(x), _ptr(w), _ptr(out), tokens, n_out, k, int(swiglu), int(PDL), int(k_split),
             _ptr(residual), _ptr(norm_weight), _ptr(sumsq_out),
             _ptr(sumsq_in), 0 if sumsq_in is None else sumsq_in.shape[1], float(norm_eps), int(norm_size),
-            _ptr(bias), float(glu_limit), float(glu_alpha), _ptr(fault), _stream(),
+            _ptr(bias), float(glu_limit), float(glu_alpha), x_pitch, int(relu2_columns), float(residual_scale), _ptr(fault),
+            _stream(),
         ),
         f"gemm_bf16({tokens}x{k} by {n_out})",
     )
@@ -1061,7 +1087,7 @@ def _row_stride(name: str, tensor: torch.Tensor) -> int:
     """Row length of a 2-D tensor whose columns are contiguous (a view of some columns is fine)."""
     if tensor.dim() != 2 or (tensor.shape[1] > 1 and tensor.stride(1) != 1):
         raise KernelError(f"{name} must be rows of contiguous columns")
-    return tensor.stride(0)
+    return tensor.stride(0) if tensor.shape[0] > 1 else max(tensor.stride(0), tensor.shape[1])
 
 
 def _state_row(state: torch.Tensor) -> tuple[int, int]:
@@ -1364,7 +1390,7 @@ def join_then_rmsnorm(x: torch.Tensor, residual: torch.Tensor, weight: torch.Ten
             or next_weight.numel() != x.shape[-1]):
         raise KernelError("join_then_rmsnorm: shapes of x, residual, the weights and out do not agree")
     _check(core().rl_add_rmsnorm(dtype_tag(x.dtype), _ptr(x), _ptr(residual), _ptr(weight), _ptr(out), None,
-                                 x.shape[0], x.shape[1], float(eps), 5, 1, None, _ptr(next_weight), int(PDL), _stream()),
+                                 x.shape[0], x.shape[1], float(eps), 5, 1, 1.0, None, _ptr(next_weight), int(PDL), _stream()),
            "join_then_rmsnorm")
     return out
 

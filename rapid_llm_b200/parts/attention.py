@@ -34,10 +34,20 @@ values are what is cached.
 
 ``qk_norm_over="row"`` norms q (and k) over the WHOLE projection at once, before it is split into heads:
 ``q <- q * rsqrt(mean(q^2) + eps) * w`` with the mean over all ``heads * head_dim`` entries and one weight per
-entry; rotation angles then come from frequencies (position kind ``rotary_frequencies``), and norm, rotation and the
-cache's store are one kernel.  ``cache_window`` says how many positions the layer's pages must keep when that differs
+entry; rotation angles then come from frequencies (position kind ``rotary_frequencies`` and its relatives), and norm,
+rotation and the cache's store are one kernel.  That path also rotates neighbouring entries together (``rotation =
+"neighbours"``) and can take the projected keys, before norm and rotation, as the values (``values_from_keys``: there is
+no value projection; the cache still holds both).  ``cache_window`` says how many positions the layer's pages must keep when that differs
 from its own ``window``: a layer whose cache another layer reads with a wider window (or without one: 0) keeps what
 that reader needs.
+
+``chunk`` cuts a sequence into chunks of so many positions, counted from position 0: a position sees the earlier ones of
+its own chunk, and the pages of a chunk go back to the pool once it is passed.  ``gate="sigmoid_head"`` multiplies head
+``h``'s output by the one number ``sigmoid(W_g x)_h``; ``o_bias`` adds a bias behind the output projection.
+
+The mixer can stand in an arrangement that stacks its sublayers' products (``first_rows`` and what follows it): its first
+product's rows and its last product's columns then lie in the arrangement's matrices, and :meth:`middle` does what is
+between the two on the columns of the stacked product's result.
 """
 
 from __future__ import annotations
@@ -99,18 +109,20 @@ class AttentionItems(StepPlanner):
 
     def __init__(self, group: int, num_kv_heads: int, head_dim: int = 0, sms: int = DEFAULT_SMS,
                  decode_clusters: dict[int, int] | None = None, tensor_core: bool = True,
-                 decode_tensor_core: bool = True) -> None:
+                 decode_tensor_core: bool = True, chunk: int = 0) -> None:
         self.group, self.num_kv_heads, self.head_dim = int(group), int(num_kv_heads), int(head_dim)
-        # decode_tensor_core False: the mixer's scores are squashed or its softmax has a sink, which the tcgen05 chunk
-        # tiles and the mma.sync tiles compute, the tcgen05 decode tiles not; tensor_core False: mma.sync tiles only
+        # decode_tensor_core False: the mixer's scores are squashed, which the tcgen05 chunk tiles and the mma.sync tiles
+        # compute, the tcgen05 decode tiles not; tensor_core False: mma.sync tiles only.  chunk: the most keys a
+        # position sees (0 = all before it), which bounds the key ranges worth having.
         self.tensor_core = bool(tensor_core)
         self.decode_tensor_core = self.tensor_core and bool(decode_tensor_core)
+        self.chunk = int(chunk)
         self.decode_clusters = dict(decode_clusters or DEFAULT_DECODE_CLUSTERS)
         # work items the kernels want in flight: two CTAs per multiprocessor, one in a decode-only
         # step, whose kernel keeps a whole multiprocessor's shared memory busy
         self.target_ctas, self.decode_target_ctas = 2 * int(sms), int(sms)
         self.key = ("attention_items", self.group, self.num_kv_heads, self.head_dim, int(sms),
-                    tuple(sorted(self.decode_clusters.items())), self.tensor_core, self.decode_tensor_core)
+                    tuple(sorted(self.decode_clusters.items())), self.tensor_core, self.decode_tensor_core, self.chunk)
 
     def capacity(self, max_tokens: int, max_entries: int) -> int:
         chunk_tiles = -(-max_tokens * self.group // kernels.CHUNK_TILE_ROWS) + max_entries
@@ -121,6 +133,11 @@ class AttentionItems(StepPlanner):
         lengths = np.asarray(shape.lengths, dtype=np.int64)
         starts = np.asarray(shape.starts, dtype=np.int64)
         rows = lengths * self.group
+        # keys before the step's first and last position of an entry, as far as its rows walk them
+        seen_first, seen_last = starts, starts + lengths
+        if self.chunk:
+            seen_first = starts % self.chunk
+            seen_last = np.minimum(seen_first + lengths, self.chunk + lengths - 1)
         is_decode = (lengths == 1) | (rows <= kernels.DECODE_TILE_ROWS)
         tensor_core = self.tensor_core and kernels.attention_tc_takes(self.head_dim, shape.page_size)
         for chunk_rows in ((kernels.CHUNK_TILE_ROWS_TC, kernels.CHUNK_TILE_ROWS) if tensor_core else (kernels.CHUNK_TILE_ROWS,)):
@@ -129,14 +146,16 @@ class AttentionItems(StepPlanner):
             ctas = int(tiles.sum()) * self.num_kv_heads
             target = self.decode_target_ctas if shape.decode_only else self.target_ctas
             splits = max(1, min(MAX_SPLITS, target // max(ctas, 1)))
+            if self.chunk:
+                splits = max(1, min(splits, -(-self.chunk // kernels.MMA_KEYS)))
             if not shape.decode_only:
-                longest = int((starts + lengths).max())
+                longest = int(seen_last.max())
                 splits = max(1, min(splits, longest // MIN_KEYS_PER_SPLIT))
             elif tensor_core and self.decode_tensor_core:
                 # ... and no more key ranges than the longest context has blocks of keys, rounded down to a power
                 # of two: a step's launch constants then change at a handful of context lengths only (the runner
                 # keeps a captured graph per set of constants)
-                blocks = max(1, -(-int((starts + lengths).max()) // kernels.DECODE_TC_KEYS))
+                blocks = max(1, -(-int(seen_last.max()) // kernels.DECODE_TC_KEYS))
                 # On long contexts the padding rows of a decode bucket do not count: their clusters come last in the
                 # grid, see one key each, and the round they add (a few microseconds) costs less than the real rows
                 # gain from more CTAs (measured at batch 5 of a bucket of 8: 5 % slower at 1,024 tokens, 10 % faster at 32,000).
@@ -161,7 +180,7 @@ class AttentionItems(StepPlanner):
         if (tensor_core and self.decode_tensor_core and not shape.decode_only and splits == 1 and chunk_rows == kernels.CHUNK_TILE_ROWS_TC
                 and bool(is_decode.any()) and not bool(is_decode.all())):
             decode_ctas = int(tiles[is_decode].sum()) * self.num_kv_heads
-            blocks = max(1, -(-int((starts + lengths)[is_decode].max()) // kernels.DECODE_TC_KEYS))
+            blocks = max(1, -(-int(seen_last[is_decode].max()) // kernels.DECODE_TC_KEYS))
             decode_splits = min(cluster_splits(decode_ctas, self.decode_clusters), 1 << (blocks.bit_length() - 1))
         entry = np.repeat(np.arange(len(lengths), dtype=np.int64), tiles)
         first = np.concatenate(([0], np.cumsum(tiles)[:-1]))
@@ -169,7 +188,7 @@ class AttentionItems(StepPlanner):
         row0 = tile_index * np.repeat(tile_rows, tiles)
         decode_tile = np.repeat(is_decode, tiles)
         # keys a tile has to walk: the tiles with the most go first, so that the last wave is short
-        keys = np.repeat(starts, tiles) + (row0 + np.repeat(tile_rows, tiles)) // self.group
+        keys = np.repeat(seen_first, tiles) + (row0 + np.repeat(tile_rows, tiles)) // self.group
 
         def items(mask: np.ndarray, ranges: int) -> np.ndarray:
             order = np.flatnonzero(mask)
@@ -215,6 +234,10 @@ class GQAAttention(Mixer):
         value_mix: str | None = None,
         qk_norm_over: str = "head",
         cache_window: int | None = None,
+        chunk: int = 0,
+        rotation: str = "halves",
+        values_from_keys: bool = False,
+        o_bias: bool = False,
         dtype,
         device,
     ) -> None:
@@ -227,10 +250,8 @@ class GQAAttention(Mixer):
         padded = -(-max(self.qk_dim, self.v_dim) // 16) * 16
         if min(self.qk_dim, self.v_dim) < 1 or padded > 256:
             raise ValueError(f"head sizes ({head_dim}, {value_dim}) must lie between 1 and 256")
-        if gate not in (None, "sigmoid"):
+        if gate not in (None, "sigmoid", "sigmoid_head"):
             raise ValueError(f"unknown output gate {gate!r}")
-        if qkv_bias and (padded != self.qk_dim or padded != self.v_dim):
-            raise ValueError("padded head sizes are not combined with a bias")
         if qk_norm_over not in ("head", "row"):
             raise ValueError(f"qk_norm_over must be 'head' or 'row', got {qk_norm_over!r}")
         self.row_norm = bool(qk_norm) and qk_norm_over == "row"
@@ -246,19 +267,26 @@ class GQAAttention(Mixer):
         self.float_prelude = self.conv_width > 0 or self.unit_after_rotation or value_mix is not None
         if self.float_prelude and (qk_norm or qkv_bias or shares_cache):
             raise ValueError("the convolution path has no weighted q/k norm, bias or shared cache")
-        if self.row_norm and qkv_bias:
-            raise ValueError("the norm over the whole projection is not combined with a bias")
+        self.neighbours, self.keys_are_values = rotation == "neighbours", bool(values_from_keys)
+        if rotation not in ("halves", "neighbours"):
+            raise ValueError(f"rotation must be 'halves' or 'neighbours', got {rotation!r}")
+        if (self.neighbours or self.keys_are_values) and not self.row_norm:
+            raise ValueError("rotation by neighbours and values taken from the keys belong to the norm over the whole projection")
+        if self.keys_are_values and (self.v_dim != self.qk_dim or shares_cache):
+            raise ValueError("values taken from the keys have the keys' size and a cache of their own")
         if not 0 <= self.conv_width <= 16 or self.softcap < 0:
             raise ValueError("conv_width must lie between 0 and 16, softcap must not be negative")
         self.names = {name: name for name in (
             "q_proj.weight", "k_proj.weight", "v_proj.weight", "o_proj.weight", "q_proj.bias", "k_proj.bias",
-            "v_proj.bias", "q_norm.weight", "k_norm.weight", "g_proj.weight", "q_conv", "k_conv", "v_conv", "sink",
+            "v_proj.bias", "o_proj.bias", "q_norm.weight", "k_norm.weight", "g_proj.weight", "q_conv", "k_conv", "v_conv", "sink",
             "value_mix")}
         self.names.update(names or {})
         self.hidden = int(hidden_size)
         self.hq, self.hkv, self.d = int(num_heads), int(num_kv_heads), padded
         self.qk_norm, self.eps = bool(qk_norm), float(qk_norm_eps)
-        self.window = int(window)
+        self.window, self.chunk = int(window), int(chunk)
+        if self.chunk < 0 or (self.chunk and (self.window or cache_window is not None)):
+            raise ValueError("chunks are not combined with a window")
         # what the pages must keep: the layer's own window, unless a reader of its cache needs more (0 = everything)
         self.cache_window = self.window if cache_window is None else int(cache_window)
         if self.cache_window < 0 or (self.cache_window and (self.window == 0 or self.cache_window < self.window)):
@@ -270,27 +298,31 @@ class GQAAttention(Mixer):
         clusters = None
         if device.type == "cuda" and dtype == torch.bfloat16:
             clusters = kernels.attention_decode_clusters(self.d, device) or None
-        plain_scores = not self.softcap and not self.has_sink
+        plain_scores = not self.softcap
         self._items = AttentionItems(self.hq // self.hkv, self.hkv, self.d, sms, clusters if plain_scores else None,
-                                     decode_tensor_core=plain_scores)
+                                     decode_tensor_core=plain_scores, chunk=self.chunk)
         self.position = POSITION_ENCODINGS.build(position, dtype=dtype, device=device)
         self.rotary_dim = int(position.params.get("rotary_dim", getattr(self.position, "rotary_dim", self.d)))
 
-        kv_rows = 0 if self.shares_cache else 2 * self.hkv * self.d
+        kv_rows = 0 if self.shares_cache else (1 if self.keys_are_values else 2) * self.hkv * self.d
         # With the norm over the whole projection the gate's rows lie behind q, k and v in ONE matrix: one product
         # reads the mixer's input once for all four, and the kernels behind it take rows wider than they use.
         self.gate_rides = bool(self.gate) and self.row_norm
         self.qkv_rows = self.hq * self.d + kv_rows
-        self.qkv = self.new_storage((self.qkv_rows + (self.hq * self.d if self.gate_rides else 0), self.hidden), MATRIX)
+        self.gate_width = 0 if not self.gate else (self.hq if self.gate == "sigmoid_head" else self.hq * self.d)
+        riding = -(-self.gate_width // 8) * 8 if self.gate_rides else 0        # rows of 16 bytes, whatever the head count
+        self.qkv = self.new_storage((self.qkv_rows + riding, self.hidden), MATRIX)
         self.o = self.new_storage((self.hidden, self.hq * self.d), MATRIX)
-        self.qkv_bias = self.new_storage((self.qkv_rows,), VECTOR) if qkv_bias else None
+        # (rows behind q, k and v that ride along have a bias of zero)
+        self.qkv_bias = self.new_storage((self.qkv.shape[0],), VECTOR) if qkv_bias else None
+        self.o_bias = self.new_storage((self.hidden,), VECTOR) if o_bias else None
         # a norm over the whole projection has a weight per laid-out entry (zero in a head's padding)
         norm_rows = (self.hq * self.d, self.hkv * self.d) if self.row_norm else (self.d, self.d)
         self.q_norm = self.new_storage((norm_rows[0],), VECTOR) if self.qk_norm else None
         self.k_norm = self.new_storage((norm_rows[1],), VECTOR) if self.qk_norm and not self.shares_cache else None
         self.g = None
         if self.gate:
-            self.g = self.qkv[self.qkv_rows :] if self.gate_rides else self.new_storage((self.hq * self.d, self.hidden), MATRIX)
+            self.g = self._riding_gate() if self.gate_rides else self.new_storage((self.gate_width, self.hidden), MATRIX)
         self.taps = self.new_storage((self.qkv_rows, self.conv_width), VECTOR) if self.conv_width > 0 else None
         self.sink = self.new_storage((self.hq,), VECTOR) if self.has_sink else None
         self.mix = self.new_storage((1,), VECTOR) if self.value_mix else None
@@ -300,8 +332,13 @@ class GQAAttention(Mixer):
                 raise ValueError("this path computes its angles from frequencies: position kind 'rotary_frequencies'")
             self.inv_freq = self.position.inv_freq
 
+    def _riding_gate(self) -> torch.Tensor:
+        return self.qkv[self.qkv_rows : self.qkv_rows + self.gate_width]
+
     # -- needs ----------------------------------------------------------------- #
     def cache_need(self) -> CacheNeed | None:
+        if self.chunk:
+            return CacheNeed("chunk", self.hkv, self.d, chunk=self.chunk)
         kind = "window" if self.cache_window > 0 else "full"
         return CacheNeed(kind, self.hkv, self.d, self.cache_window)
 
@@ -324,9 +361,12 @@ class GQAAttention(Mixer):
         }
         if not self.shares_cache:
             specs["k_proj.weight"] = TensorSpec((self.hkv * self.qk_dim, self.hidden))
-            specs["v_proj.weight"] = TensorSpec((self.hkv * self.v_dim, self.hidden))
+            if not self.keys_are_values:
+                specs["v_proj.weight"] = TensorSpec((self.hkv * self.v_dim, self.hidden))
+        if self.o_bias is not None:
+            specs["o_proj.bias"] = TensorSpec((self.hidden,), VECTOR)
         if self.qkv_bias is not None:
-            for name in ("q_proj", "k_proj", "v_proj")[: 1 if self.shares_cache else 3]:
+            for name in ("q_proj", "k_proj", "v_proj")[: 1 if self.shares_cache else 2 if self.keys_are_values else 3]:
                 specs[f"{name}.bias"] = TensorSpec((specs[f"{name}.weight"].shape[0],), VECTOR)
         if self.qk_norm:
             q_count, k_count = (self.hq * self.qk_dim, self.hkv * self.qk_dim) if self.row_norm else (self.qk_dim, self.qk_dim)
@@ -334,7 +374,7 @@ class GQAAttention(Mixer):
             if not self.shares_cache:
                 specs["k_norm.weight"] = TensorSpec((k_count,), VECTOR, init="ones_normal")
         if self.gate:
-            specs["g_proj.weight"] = TensorSpec((self.hq * self.v_dim, self.hidden))
+            specs["g_proj.weight"] = TensorSpec((self.hq if self.gate == "sigmoid_head" else self.hq * self.v_dim, self.hidden))
         if self.conv_width > 0:
             specs["q_conv"] = TensorSpec((self.hq * self.qk_dim, self.conv_width), VECTOR)
             specs["k_conv"] = TensorSpec((self.hkv * self.qk_dim, self.conv_width), VECTOR)
@@ -363,14 +403,20 @@ class GQAAttention(Mixer):
         elif name == "o_proj.weight":
             self.o.view(self.hidden, self.hq, self.d)[:, :, : self.v_dim].copy_(
                 tensor.view(self.hidden, self.hq, self.v_dim))
+        elif name == "g_proj.weight" and self.gate == "sigmoid_head":
+            self.g.copy_(tensor)
         elif name == "g_proj.weight":
             self._heads(self.g, self.hq)[:, : self.v_dim].copy_(tensor.view(self.hq, self.v_dim, -1))
         elif name == "q_proj.bias":
-            self.qkv_bias[:q_rows].copy_(tensor.to(torch.float32))
+            self.qkv_bias[:q_rows].view(self.hq, self.d)[:, : self.qk_dim].copy_(tensor.to(torch.float32).view(self.hq, -1))
         elif name == "k_proj.bias":
-            self.qkv_bias[q_rows : q_rows + kv_rows].copy_(tensor.to(torch.float32))
+            self.qkv_bias[q_rows : q_rows + kv_rows].view(self.hkv, self.d)[:, : self.qk_dim].copy_(
+                tensor.to(torch.float32).view(self.hkv, -1))
         elif name == "v_proj.bias":
-            self.qkv_bias[q_rows + kv_rows :].copy_(tensor.to(torch.float32))
+            self.qkv_bias[q_rows + kv_rows : self.qkv_rows].view(self.hkv, self.d)[:, : self.v_dim].copy_(
+                tensor.to(torch.float32).view(self.hkv, -1))
+        elif name == "o_proj.bias":
+            self.o_bias.copy_(tensor.to(torch.float32))
         elif name == "q_conv":
             self._heads(self.taps[:q_rows], self.hq)[:, : self.qk_dim].copy_(tensor.to(torch.float32).view(self.hq, self.qk_dim, -1))
         elif name == "k_conv":
@@ -396,13 +442,13 @@ class GQAAttention(Mixer):
 
     def parameter_bytes(self) -> int:
         total = (self.qkv.numel() + self.o.numel() + (0 if self.g is None or self.gate_rides else self.g.numel())) * self.qkv.element_size()
-        for vector in (self.q_norm, self.k_norm, self.qkv_bias, self.taps, self.sink, self.mix):
+        for vector in (self.q_norm, self.k_norm, self.qkv_bias, self.o_bias, self.taps, self.sink, self.mix):
             if vector is not None:
                 total += vector.numel() * 4
         return total
 
     def workspace_elements_per_token(self) -> int:
-        gate = 2 * self.hq * self.d if self.gate else 0
+        gate = self.gate_width + self.hq * self.d if self.gate else 0
         return self.qkv.shape[0] + 2 * self.hq * self.d + self.hidden + gate      # qkv, q, attended, projected
 
     def uses_libraries(self) -> set[str]:
@@ -414,15 +460,31 @@ class GQAAttention(Mixer):
 
     # -- forward --------------------------------------------------------------- #
     def forward(self, x, batch, cache, then_norm=None):
+        rows = x.shape[0]
+        qkv = batch.workspace.get("attn_qkv", rows, self.qkv.shape[0], x.dtype)
+        gemm.linear(x, self.qkv, qkv, batch.fault, bias=self.qkv_bias, defer=batch.defer_products)
+        attended = self._attended(qkv, batch, cache)
+        if self.gate:
+            if self.gate_rides:
+                gate = qkv[:, self.qkv_rows : self.qkv_rows + self.gate_width]          # the first product brought it along
+            else:
+                gate = batch.workspace.get("attn_gate", rows, self.gate_width, x.dtype)
+                gemm.linear(x, self.g, gate, batch.fault)
+            gated = batch.workspace.get("attn_gated", rows, self.hq * self.d, x.dtype)
+            attended = kernels.sigmoid_gate(attended, gate, gated)
+        out = batch.workspace.get("attn_proj", rows, self.hidden, x.dtype)
+        return gemm.linear(attended, self.o, out, batch.fault, then_norm=then_norm, bias=self.o_bias, defer=batch.defer_products)
+
+    def _attended(self, qkv, batch, cache) -> torch.Tensor:
+        """From the first product's result to the heads side by side, before the gate: norms, rotation, the cache's
+        store and attention."""
         if cache.group is None or cache.pages is None:
             raise ValueError("attention needs a cache group; the engine did not give this layer one")
         if cache.writes == self.shares_cache:
             raise ValueError("the layer's cache role in the run order does not match shares_cache")
         group = batch.groups[cache.group]
-        rows = x.shape[0]
-        qkv = batch.workspace.get("attn_qkv", rows, self.qkv.shape[0], x.dtype)
-        gemm.linear(x, self.qkv, qkv, batch.fault, bias=self.qkv_bias, defer=batch.defer_products)
-        q = batch.workspace.get("attn_q", rows, self.hq * self.d, x.dtype)
+        rows = qkv.shape[0]
+        q = batch.workspace.get("attn_q", rows, self.hq * self.d, qkv.dtype)
         if self.float_prelude:
             self._float_prelude(qkv, q, batch, cache, group)
         elif self.row_norm:
@@ -431,21 +493,38 @@ class GQAAttention(Mixer):
                 k_weight=self.k_norm, q_count=self.hq * self.qk_dim, k_count=self.hkv * self.qk_dim,
                 inv_freq=self.inv_freq, positions=batch.positions, eps=self.eps, fault=batch.fault,
                 kv_dest=group.kv_dest if cache.writes else None, cache=cache.pages if cache.writes else None,
-                page_size=group.page_size)
+                page_size=group.page_size, neighbours=self.neighbours, values_are_keys=self.keys_are_values)
         else:
             self._norm_rope_write(qkv, q, batch, cache, group)
-        attended = batch.workspace.get("attn_out", rows, self.hq * self.d, x.dtype)
+        attended = batch.workspace.get("attn_out", rows, self.hq * self.d, qkv.dtype)
         self.attend(q, cache.pages, attended, batch, group)
-        if self.gate:
-            if self.gate_rides:
-                gate = qkv[:, self.qkv_rows :]          # the first product brought it along
-            else:
-                gate = batch.workspace.get("attn_gate", rows, self.hq * self.d, x.dtype)
-                gemm.linear(x, self.g, gate, batch.fault)
-            gated = batch.workspace.get("attn_gated", rows, self.hq * self.d, x.dtype)
-            attended = kernels.sigmoid_gate(attended, gate, gated)
-        out = batch.workspace.get("attn_proj", rows, self.hidden, x.dtype)
-        return gemm.linear(attended, self.o, out, batch.fault, then_norm=then_norm, defer=batch.defer_products)
+        return attended
+
+    # -- in an arrangement that stacks its sublayers' products ------------------- #
+    @property
+    def stacks(self) -> bool:
+        return self.gate_rides and not self.float_prelude
+
+    @property
+    def first_rows(self) -> int:
+        return self.qkv.shape[0]
+
+    @property
+    def last_columns(self) -> int:
+        return self.hq * self.d
+
+    def adopt(self, first, first_bias, last) -> None:
+        """Keep the weights of the first and the last product in the arrangement's matrices (views) from here on."""
+        self.qkv, self.o = first, last
+        self.g = self._riding_gate()
+        if self.qkv_bias is not None:
+            self.qkv_bias = first_bias
+
+    def middle(self, wide, batch, cache) -> None:
+        """``wide [T, first_rows]``, the first product's result (a view of some columns of wider rows), in; the last
+        product's input in its first ``last_columns`` columns, out: the gated heads take the queries' place."""
+        attended = self._attended(wide, batch, cache)
+        kernels.sigmoid_gate(attended, wide[:, self.qkv_rows : self.qkv_rows + self.gate_width], wide[:, : self.last_columns])
 
     def _float_prelude(self, qkv, q, batch, cache, group) -> None:
         """Projection -> short convolution (float32, the slot's tail before the step's rows) -> rotation ->
@@ -502,12 +581,12 @@ class GQAAttention(Mixer):
                 block_table=group.block_table, num_heads=self.hq, num_kv_heads=self.hkv, head_dim=self.d,
                 window=self.window, scale=self.scale, fault=batch.fault, decode_rows=plan.get("decode_rows", 0),
                 chunk_rows=plan.get("chunk_rows", kernels.CHUNK_TILE_ROWS),
-                decode_splits=plan.get("decode_splits", 0), softcap=self.softcap, sink=self.sink,
+                decode_splits=plan.get("decode_splits", 0), softcap=self.softcap, sink=self.sink, chunk=self.chunk,
             )
             return
         kernels.attention_generic(
             q, pages, out,
             positions=batch.positions, token_slot=batch.token_slot, block_table=group.block_table,
             num_heads=self.hq, num_kv_heads=self.hkv, head_dim=self.d,
-            window=self.window, scale=self.scale, fault=batch.fault, softcap=self.softcap, sink=self.sink,
+            window=self.window, scale=self.scale, fault=batch.fault, softcap=self.softcap, sink=self.sink, chunk=self.chunk,
         )

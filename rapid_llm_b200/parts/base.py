@@ -10,7 +10,7 @@ seam through factory methods and class flags on the model skeleton
 Roles and what each must provide:
 
 * **Mixer** — ``forward(x, batch, cache) -> y`` over the packed tokens of a step;
-  ``cache_need()`` says which pages it wants (all keys, a window of them, none),
+  ``cache_need()`` says which pages it wants (all keys, a window or a chunk of them, none),
   ``state_need()`` which per-request state of fixed size, and ``step_planner()`` may name
   host-side planning it wants done once per step (work lists for its kernels).
 * **FeedForward** — ``forward(x, batch) -> y``.
@@ -57,8 +57,9 @@ class TensorSpec:
 class CacheNeed:
     """Pages a mixer wants.
 
-    ``kind`` says which positions are kept: ``"full"`` (all of them) or ``"window"`` (the last
-    ``window``).  What a page holds is the mixer's business: by default a key and a value per kv
+    ``kind`` says which positions are kept: ``"full"`` (all of them), ``"window"`` (the last
+    ``window``) or ``"chunk"`` (those of the chunk of ``chunk`` positions, counted from position 0, that the next
+    position lies in).  What a page holds is the mixer's business: by default a key and a value per kv
     head, ``[2, num_kv_heads, page_size, head_dim]``; a mixer that caches something else (one
     latent row per token, keys without values) names the shape of one token's row in
     ``token_shape`` and gets pages ``[page_size, *token_shape]``.
@@ -69,9 +70,10 @@ class CacheNeed:
     head_dim: int = 0
     window: int = 0
     token_shape: tuple[int, ...] | None = None
+    chunk: int = 0
 
     def group_key(self) -> tuple:
-        return (self.kind, self.window, self.num_kv_heads, self.head_dim, self.token_shape)
+        return (self.kind, self.window, self.chunk, self.num_kv_heads, self.head_dim, self.token_shape)
 
     def page_shape(self, page_size: int) -> tuple[int, ...]:
         if self.token_shape is not None:
@@ -191,6 +193,11 @@ class Mixer(Part):
     # product may take along, returning ``ScaledRows`` instead of a tensor.  Without the flag a
     # part sees plain tensors only.
     rides_norms = False
+    # A mixer or feed-forward with ``stacks`` can stand in an arrangement that runs the sublayers' first products as one
+    # and their last products as one: ``first_rows`` output rows of the first product and ``last_columns`` inputs of the
+    # last are its own, ``adopt`` moves its weights into views of the arrangement's matrices, and ``middle`` (a mixer)
+    # turns its columns of the first product's result into the last product's input, in place.
+    stacks = False
 
     def cache_need(self) -> CacheNeed | None:
         return None
@@ -207,6 +214,7 @@ class Mixer(Part):
 
 class FeedForward(Part):
     rides_norms = False      # as for a mixer
+    stacks = False           # as for a mixer
 
     def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
         raise NotImplementedError
@@ -245,6 +253,10 @@ class Block(Part):
     # True for an arrangement that keeps the whole stream in ``residual`` (float32) and hands on, as ``x``, only its
     # rounding to the engine's dtype: the model then norms ``residual`` alone at the end, not ``x + residual``.
     stream_in_residual = False
+
+    # True for an arrangement that takes ``x = None`` as "the stream is complete, nothing is waiting to join it": what the
+    # model hands the first layer when the embedding has opened the float32 stream itself.
+    takes_open_stream = False
 
     def leading_norm(self) -> "Norm | None":
         """The norm this block starts with, if the block takes its unscaled result

@@ -18,6 +18,9 @@ sublayers read the stream itself; the stream is the float32 ``residual`` and ``x
 
 ``postnorm`` (:class:`PostNormBlock`): the norm behind the sum, ``h' = Norm(alpha h + Mixer(h));
 h'' = Norm(alpha h' + FeedForward(h'))``; the stream is the norm's own result, float32 in ``residual``.
+
+``shared_norm`` (:class:`SharedNormBlock`): one norm in front of both sublayers, ``h' = h + m (Mixer(n) + FeedForward(n))``
+with ``n = Norm(h)``; the two sublayers' first products are one product, and so are their last.
 """
 
 from __future__ import annotations
@@ -27,13 +30,15 @@ import torch
 from ..config.model_spec import LayerSpec
 from ..ops import gemm, kernels
 from ..ops.gemm import ScaledRows
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, TensorSpec
+from .base import BLOCKS, FEED_FORWARDS, MATRIX, MIXERS, NORMS, VECTOR, Block, TensorSpec
 from .norm import ADD, FIRST
 
 
 @BLOCKS.register("prenorm")
 class PreNormBlock(Block):
     """``names`` maps the roles to their checkpoint sub-prefixes."""
+
+    takes_open_stream = True
 
     NAMES = {
         "mixer_norm": "input_layernorm.",
@@ -106,18 +111,7 @@ class PreNormBlock(Block):
 
     def forward(self, x, residual, batch, cache, then_norm=None, addend=None):
         """``(x, residual)`` in, ``(x, residual)`` out; ``residual`` is ``None`` for the first layer."""
-        if not self.mixer_norm.reads_deferred:
-            gemm.flush()        # a norm that is no kernel of ops.kernels reads finished results only
-        extra = {} if addend is None else {"addend": addend}
-        if isinstance(x, ScaledRows):
-            if addend is not None:
-                raise ValueError("a norm that rode on the product before it cannot take an addend")
-            normed = x          # the block before took this block's first norm along
-        elif residual is None:
-            residual = batch.workspace.get("residual", x.shape[0], x.shape[1], torch.float32)
-            normed = self.mixer_norm.forward(x, residual, batch, mode=FIRST, write_residual=True, **extra)
-        else:
-            normed = self.mixer_norm.forward(x, residual, batch, mode=ADD, write_residual=True, **extra)
+        normed, residual = self._lead(x, residual, batch, addend)
         if self.feed_forward is None:
             if self.mixer.rides_norms:
                 offer = then_norm.following(residual, batch) if then_norm is not None else None
@@ -139,6 +133,27 @@ class PreNormBlock(Block):
             return self.feed_forward.forward(normed, batch, then_norm=offer), residual
         return self.feed_forward.forward(normed, batch), residual
 
+    def _lead(self, x, residual, batch, addend):
+        """The block's first norm of the stream: ``(normed rows, residual)``.  ``x`` is what still has to join the stream
+        (``None``: nothing, the stream is complete; ``residual`` ``None``: ``x`` opens it)."""
+        if not self.mixer_norm.reads_deferred:
+            gemm.flush()        # a norm that is no kernel of ops.kernels reads finished results only
+        extra = {} if addend is None else {"addend": addend}
+        if x is None:
+            if addend is not None:
+                raise ValueError("a stream that the embedding opened takes no addend")
+            return self.mixer_norm.of_stream(residual, batch), residual
+        if isinstance(x, ScaledRows):
+            if addend is not None:
+                raise ValueError("a norm that rode on the product before it cannot take an addend")
+            normed = x          # the block before took this block's first norm along
+        elif residual is None:
+            residual = batch.workspace.get("residual", x.shape[0], x.shape[1], torch.float32)
+            normed = self.mixer_norm.forward(x, residual, batch, mode=FIRST, write_residual=True, **extra)
+        else:
+            normed = self.mixer_norm.forward(x, residual, batch, mode=ADD, write_residual=True, **extra)
+        return normed, residual
+
 
 @BLOCKS.register("outnorm")
 class OutputNormBlock(PreNormBlock):
@@ -150,6 +165,7 @@ class OutputNormBlock(PreNormBlock):
     rides on one."""
 
     stream_in_residual = True
+    takes_open_stream = False
 
     def leading_norm(self):
         return None
@@ -197,6 +213,7 @@ class SandwichBlock(PreNormBlock):
     of the next sublayer (of this block, or of the next block if that is a sandwich block too)."""
 
     stream_in_residual = True
+    takes_open_stream = False
     NAMES = {"mixer_norm": "norm1", "mixer_out_norm": "norm1b", "mixer": "mix.", "feed_forward_norm": "norm2",
              "feed_forward_out_norm": "norm2b", "feed_forward": "mlp."}
 
@@ -268,6 +285,7 @@ class PostNormBlock(PreNormBlock):
     (``layernorm``)."""
 
     stream_in_residual = True
+    takes_open_stream = False
     NAMES = {"mixer_norm": "norm1", "mixer": "mix.", "feed_forward_norm": "norm2", "feed_forward": "mlp."}
 
     def __init__(self, *, layer: LayerSpec, dtype, device, names: dict[str, str] | None = None) -> None:
@@ -299,3 +317,66 @@ class PostNormBlock(PreNormBlock):
                 gemm.flush()
                 x = self.feed_forward_norm.post_join(wide, residual, self.alpha, batch)
         return x, residual
+
+
+@BLOCKS.register("shared_norm")
+class SharedNormBlock(PreNormBlock):
+    """One norm in front of both sublayers, whose results join the stream together:
+    ``h <- h + m * (Mixer(n) + FeedForward(n))``, ``n = Norm(h)``.  The weight ``m`` is the norms' ``add_scale`` (as in
+    ``prenorm``, the sum waits for the next norm, or rides on the last product with it).
+
+    Both sublayers read the same rows and their results are summed, so where both can (``stacks``) their weights lie
+    in two matrices and the layer has two products: ``[W_ff1; W_mix1] n``, whose columns the sublayers work on in place,
+    and ``[W_ff2 | W_mix2]`` on the columns they leave, which forms the sum of the sublayers in its float32 accumulator.
+    The input is read once, the sum is rounded once, and a small step has two weight streams instead of four."""
+
+    NAMES = {"mixer_norm": "norm1", "mixer": "mix.", "feed_forward": "mlp."}
+
+    def __init__(self, *, layer: LayerSpec, dtype, device, names: dict[str, str] | None = None) -> None:
+        super().__init__(layer=layer, dtype=dtype, device=device, names=names)
+        self.feed_forward_norm = None
+        mixer, ff = self.mixer, self.feed_forward
+        self.stacked = getattr(mixer, "stacks", False) and (ff is None or getattr(ff, "stacks", False))
+        if not self.stacked:
+            return
+        # the feed-forward first: all its columns stay, so the last product's input is one run of columns
+        self.ff_columns = 0 if ff is None else ff.first_rows
+        self.hidden = mixer.hidden
+        self.first = self.new_storage((self.ff_columns + mixer.first_rows, self.hidden), MATRIX)
+        self.first_bias = self.new_storage((self.first.shape[0],), VECTOR) if mixer.qkv_bias is not None else None
+        self.last = self.new_storage((self.hidden, self.ff_columns + mixer.last_columns), MATRIX)
+        if ff is not None:
+            ff.adopt(self.first[: self.ff_columns], self.last[:, : self.ff_columns])
+        mixer.adopt(self.first[self.ff_columns :], None if self.first_bias is None else self.first_bias[self.ff_columns :],
+                    self.last[:, self.ff_columns :])
+
+    def _children(self):
+        children = [(self.names["mixer_norm"], self.mixer_norm), (self.names["mixer"], self.mixer)]
+        if self.feed_forward is not None:
+            children.append((self.names["feed_forward"], self.feed_forward))
+        return tuple(children)
+
+    def leading_norm(self):
+        return self.mixer_norm if self.stacked else None
+
+    def uses_libraries(self) -> set[str]:
+        return super().uses_libraries() | (set() if self.stacked or self.feed_forward is None else {"recurrent"})
+
+    def forward(self, x, residual, batch, cache, then_norm=None, addend=None):
+        normed, residual = self._lead(x, residual, batch, addend)
+        rows, space = normed.shape[0], batch.workspace
+        if not self.stacked:
+            mixed = self.mixer.forward(normed, batch, cache)
+            gemm.flush()
+            if self.feed_forward is None:
+                return mixed, residual
+            wide = self.feed_forward.forward(normed, batch)
+            gemm.flush()
+            return kernels.scaled_sum(mixed, wide, 1.0, 1.0, space.get("shared_sum", rows, mixed.shape[1], mixed.dtype)), residual
+        wide = space.get("shared_wide", rows, self.first.shape[0], normed.dtype)
+        gemm.linear(normed, self.first, wide, batch.fault, bias=self.first_bias, relu2_columns=self.ff_columns)
+        self.mixer.middle(wide[:, self.ff_columns :], batch, cache)
+        offer = then_norm.following(residual, batch) if then_norm is not None else None
+        out = space.get("shared_out", rows, self.hidden, normed.dtype)
+        return gemm.linear(wide[:, : self.last.shape[1]], self.last, out, batch.fault, then_norm=offer,
+                           bias=self.mixer.o_bias), residual

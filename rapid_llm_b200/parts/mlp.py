@@ -86,8 +86,8 @@ class ClampedGLU(SwiGLU):
         return gemm.linear(act, self.down, batch.workspace.get("ffn_out", rows, self.hidden, x.dtype), batch.fault)
 
 
-# activation name -> (number of learned scalars, kernel over [T, I] rows)
-ACTIVATIONS = {"xielu": (2, kernels.xielu)}
+# activation name -> (number of learned scalars, kernel over [T, I] rows, library it lives in)
+ACTIVATIONS = {"xielu": (2, kernels.xielu, "recurrent"), "relu_squared": (0, kernels.relu_squared, "core")}
 
 
 @FEED_FORWARDS.register("dense")
@@ -96,6 +96,8 @@ class DenseFeedForward(FeedForward):
 
     ``xielu``: with the two scalars ``p, q`` of the activation's tensor, ``z > 0: softplus(p) z^2 + z / 2`` and
     ``z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2`` (float32 arithmetic on the product's result).
+    ``relu_squared``: ``max(z, 0)^2``, no scalars; it rides in the first product's epilogue where the tensor-core product
+    runs, and in an arrangement that stacks its sublayers' products this feed-forward can be the stack's first part.
     """
 
     def __init__(self, *, hidden_size: int, intermediate_size: int, activation: str, dtype, device,
@@ -107,15 +109,15 @@ class DenseFeedForward(FeedForward):
         self.names = (up_name, down_name, act_name)
         self.up = self.new_storage((self.inter, self.hidden), MATRIX)
         self.down = self.new_storage((self.hidden, self.inter), MATRIX)
-        self.scalars = self.new_storage((ACTIVATIONS[activation][0],), VECTOR)
+        count = ACTIVATIONS[activation][0]
+        self.scalars = self.new_storage((count,), VECTOR) if count else None
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         up, down, act = self.names
-        return {
-            up: TensorSpec((self.inter, self.hidden)),
-            down: TensorSpec((self.hidden, self.inter)),
-            act: TensorSpec(tuple(self.scalars.shape), VECTOR),
-        }
+        specs = {up: TensorSpec((self.inter, self.hidden)), down: TensorSpec((self.hidden, self.inter))}
+        if self.scalars is not None:
+            specs[act] = TensorSpec(tuple(self.scalars.shape), VECTOR)
+        return specs
 
     def load_tensor(self, name: str, tensor: torch.Tensor) -> None:
         up, down, act = self.names
@@ -123,25 +125,44 @@ class DenseFeedForward(FeedForward):
             self.up.copy_(tensor)
         elif name == down:
             self.down.copy_(tensor)
-        elif name == act:
+        elif name == act and self.scalars is not None:
             self.scalars.copy_(tensor.to(torch.float32))
         else:
             raise KeyError(name)
 
     def parameter_bytes(self) -> int:
-        return (self.up.numel() + self.down.numel()) * self.up.element_size() + self.scalars.numel() * 4
+        return (self.up.numel() + self.down.numel()) * self.up.element_size() + (0 if self.scalars is None else self.scalars.numel() * 4)
 
     def workspace_elements_per_token(self) -> int:
         return 2 * self.inter + self.hidden
 
     def uses_libraries(self) -> set[str]:
-        return {"recurrent"} | ({"gemm"} if self.dtype == torch.bfloat16 else set())
+        return {ACTIVATIONS[self.activation][2]} | ({"gemm"} if self.dtype == torch.bfloat16 else set())
 
     def forward(self, x, batch):
         rows = x.shape[0]
         wide = batch.workspace.get("ffn_up", rows, self.inter, x.dtype)
-        gemm.linear(x, self.up, wide, batch.fault)
-        act = batch.workspace.get("ffn_act", rows, self.inter, x.dtype)
-        ACTIVATIONS[self.activation][1](wide, act, self.scalars)
+        if self.activation == "relu_squared":
+            act = gemm.linear(x, self.up, wide, batch.fault, relu2_columns=self.inter)
+        else:
+            gemm.linear(x, self.up, wide, batch.fault)
+            act = batch.workspace.get("ffn_act", rows, self.inter, x.dtype)
+            ACTIVATIONS[self.activation][1](wide, act, self.scalars)
         out = batch.workspace.get("ffn_out", rows, self.hidden, x.dtype)
         return gemm.linear(act, self.down, out, batch.fault)
+
+    # -- in an arrangement that stacks its sublayers' products ------------------- #
+    @property
+    def stacks(self) -> bool:
+        return self.activation == "relu_squared"
+
+    @property
+    def first_rows(self) -> int:
+        return -(-self.inter // 8) * 8       # rows behind the true ones are zeros, and zeros stay zeros
+
+    last_columns = first_rows                # every column of the first product is one of the last product's input
+
+    def adopt(self, first, last) -> None:
+        """Keep the weights of the two products in the arrangement's matrices (views) from here on; the arrangement's
+        first product applies the activation to all :attr:`first_rows` columns."""
+        self.up, self.down = first[: self.inter], last[:, : self.inter]

@@ -21,10 +21,12 @@ FIRST, ADD, PLAIN = 0, 1, 2
 class RMSNorm(Norm):
     reads_deferred = True       # it launches through ops.kernels, which runs queued products first
 
-    def __init__(self, *, size: int, eps: float, dtype, device, name: str = "weight", unit_offset: bool = False) -> None:
+    def __init__(self, *, size: int, eps: float, dtype, device, name: str = "weight", unit_offset: bool = False,
+                 add_scale: float = 1.0) -> None:
         super().__init__(dtype=dtype, device=device)
         self.size = int(size)
         self.eps = float(eps)
+        self.add_scale = float(add_scale)      # weighs what joins the stream in front of this norm (mode ADD)
         self.name = name          # the tensor's name after the part's prefix (may be empty)
         self.unit_offset = bool(unit_offset)
         self.weight = self.new_storage((self.size,), VECTOR)
@@ -49,7 +51,7 @@ class RMSNorm(Norm):
         """This norm of ``residual + (a product's result)``, as an offer to that product."""
         if self.dtype != torch.bfloat16 or residual is None:
             return None
-        return gemm.FollowingNorm(residual, self.weight, self.eps, batch.workspace)
+        return gemm.FollowingNorm(residual, self.weight, self.eps, batch.workspace, self.add_scale)
 
     def join(self, y, residual, batch, name="stream_rows"):
         """The norm on a sublayer's output: ``residual += norm(y)`` in float32; returns the new stream in the
@@ -69,7 +71,7 @@ class RMSNorm(Norm):
         return kernels.stream_rmsnorm(residual, self.weight, out, self.eps, row_index)
 
     def forward(self, x, residual, batch, *, mode, write_residual, row_index=None, name="normed", addend=None):
-        """Norm of ``x`` (``FIRST``/``PLAIN``) or of ``x + residual`` (``ADD``).
+        """Norm of ``x`` (``FIRST``/``PLAIN``) or of ``add_scale * x + residual`` (``ADD``).
 
         With ``write_residual`` the float32 sum is stored into ``residual``.  ``row_index``
         selects input rows (the rows whose logits are wanted, for the final norm).  ``addend``
@@ -82,6 +84,7 @@ class RMSNorm(Norm):
             mode=mode, write_residual=write_residual, row_index=row_index,
             extra_rows=None if addend is None else addend.rows,
             extra_vector=None if addend is None else addend.vector,
+            x_scale=self.add_scale,
         )
 
 

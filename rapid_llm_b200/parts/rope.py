@@ -75,6 +75,24 @@ class RotaryFrequencies(PositionEncoding):
         raise ValueError("this position encoding has no tables; its kernel computes the angles")
 
 
+@POSITION_ENCODINGS.register("banded_frequencies")
+class BandedFrequencies(RotaryFrequencies):
+    """Frequencies stretched by the length of their wave (the rule of Llama 3.1).  With ``wave = 2 pi / f``: ``f`` stays
+    where ``wave < original / high``, becomes ``f / factor`` where ``wave > original / low``, and in between moves from
+    one to the other, ``(1 - s) f / factor + s f`` with ``s = (original / wave - low) / (high - low)``."""
+
+    def __init__(self, *, rotary_dim: int, theta: float, max_positions: int, factor: float, low: float, high: float,
+                 original: float, dtype, device) -> None:
+        super().__init__(rotary_dim=rotary_dim, theta=theta, max_positions=max_positions, dtype=dtype, device=device)
+        if not factor > 0 or not original > 0 or not 0 < low <= high:
+            raise ValueError(f"the bands need 0 < low <= high and a positive factor and original, got {low}, {high}, {factor}, {original}")
+        plain = float(theta) ** -(torch.arange(0, self.rotary_dim, 2, dtype=torch.float64) / max(self.rotary_dim, 1))
+        turns = float(original) * plain / (2.0 * torch.pi)         # original / wave
+        span = float(high) - float(low)
+        share = ((turns - float(low)) / span).clamp(0.0, 1.0) if span > 0 else (turns >= float(high)).to(torch.float64)
+        self.inv_freq = ((1.0 - share) * plain / float(factor) + share * plain).to(torch.float32).to(self.device)
+
+
 @POSITION_ENCODINGS.register("yarn_frequencies")
 class YarnFrequencies(RotaryFrequencies):
     """Frequencies stretched for contexts longer than the ``original`` one: the slow ones divided by ``factor``, the
