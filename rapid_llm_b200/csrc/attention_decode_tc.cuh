@@ -76,6 +76,9 @@ struct DecodeTcArgs {
   int hq, hkv, page_size, num_pages, max_pages, slots, window, chunk, splits;
   int cluster_merge;        // the CTAs of an item's splits are one cluster and merge among themselves
   float scale_log2;
+  int out_stride;           // elements from a token's row of out to the next
+  const bf16* gate;         // [tokens, hq] or null: a head's output is multiplied by sigmoid(gate)
+  int gate_stride;
   const float* sink;        // [hq] float32 or null: exp(sink[head]) joins every row's denominator once
   int* fault;
 };
@@ -474,18 +477,19 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
       const float value = out_acc[n] * w0 + exchange[n * 128 + t] * w1;
       float inv = total > 0.0f ? 1.0f / total : 0.0f;
       const float lse = total > 0.0f ? m + log2f(total) : -INFINITY;
-      const int p = row0 + n, token = p / group;
-      const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group + (p - token * group);
+      const int p = row0 + n, token = p / group, head = kv_head * group + (p - token * group);
+      const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + head;
       if (args.sink != nullptr && args.splits == 1) {
         // an unsplit row's denominator takes the sink here; a split one's where its parts meet
-        const float sink2 = args.sink[row % args.hq] * 1.4426950408889634f;
+        const float sink2 = args.sink[head] * 1.4426950408889634f;
         const float top = fmaxf(m, sink2);
         const float keys = m == -INFINITY ? 0.0f : fast_exp2(m - top);
         inv = keys / (total * keys + fast_exp2(sink2 - top));
       }
+      if (args.splits == 1) inv *= head_gate(args.gate, args.gate_stride, tok_begin + token, head);
       const float merged = value * inv;
       if (args.splits == 1) {
-        args.out[row * kTcD + t] = __float2bfloat16_rn(merged);
+        args.out[static_cast<size_t>(tok_begin + token) * args.out_stride + head * kTcD + t] = __float2bfloat16_rn(merged);
       } else if (args.cluster_merge) {
         split_out[n * 128 + t] = merged;
         if (t == 0) split_lse[n] = lse;
@@ -531,9 +535,9 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
             }
           }
         }
-        const int p = row0 + n, token = p / group;
-        const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group + (p - token * group);
-        const float sink2 = args.sink != nullptr ? args.sink[row % args.hq] * 1.4426950408889634f : -INFINITY;
+        const int p = row0 + n, token = p / group, head = kv_head * group + (p - token * group);
+        const float sink2 = args.sink != nullptr ? args.sink[head] * 1.4426950408889634f : -INFINITY;
+        const float factor = head_gate(args.gate, args.gate_stride, tok_begin + token, head);
         float m = sink2;
 #pragma unroll
         for (int r = 0; r < 8; ++r) m = fmaxf(m, lse_of[r]);
@@ -561,7 +565,8 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
             }
           }
         }
-        args.out[row * kTcD + t] = __float2bfloat16_rn(total > 0.0f ? value / total : 0.0f);
+        args.out[static_cast<size_t>(tok_begin + token) * args.out_stride + head * kTcD + t] =
+            __float2bfloat16_rn(total > 0.0f ? value / total * factor : 0.0f);
       }
     }
     __syncwarp();

@@ -26,7 +26,9 @@ template <typename T, int kMaxD>
 __global__ void attention_generic_kernel(
     const T* __restrict__ q,            // [tokens, hq, d]
     const T* __restrict__ cache,        // [num_pages, kv_planes (2, or 1: values are the keys' rows), hkv, page_size, d]
-    T* __restrict__ out,                // [tokens, hq, d]
+    T* out,                             // [tokens, hq, d], rows out_stride apart
+    int out_stride,
+    const T* gate, int gate_stride,     // [tokens, hq] or null: head outputs are multiplied by its sigmoid
     const int* __restrict__ positions,  // [tokens]
     const int* __restrict__ token_slot, // [tokens]
     const int* __restrict__ block_table,  // [slots, max_pages]
@@ -41,7 +43,7 @@ __global__ void attention_generic_kernel(
   const int kv_head = head / (hq / hkv);
   const int pos = positions[t];
   const int slot = token_slot[t];
-  T* o = out + (static_cast<size_t>(t) * hq + head) * d;
+  T* o = out + static_cast<size_t>(t) * out_stride + static_cast<size_t>(head) * d;
   if (slot < 0 || slot >= slots || pos < 0 || pos >= max_pages * page_size) {
     if (lane == 0) atomicOr(fault, slot < 0 || slot >= slots ? kFaultSlot : kFaultPosition);
     for (int i = lane; i < d; i += 32) o[i] = from_float<T>(0.0f);
@@ -118,6 +120,7 @@ __global__ void attention_generic_kernel(
     const float keys = running_max == -INFINITY ? 0.0f : expf(running_max - top);
     inv_sum = keys / (running_sum * keys + expf(s - top));
   }
+  inv_sum *= head_gate(gate, gate_stride, t, head);
 #pragma unroll
   for (int i = 0; i < kMaxD / 32; ++i) {
     const int col = lane + 32 * i;
@@ -127,7 +130,8 @@ __global__ void attention_generic_kernel(
 
 }  // namespace rl
 
-extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache, void* out,
+extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache, void* out, int out_stride,
+                                    const void* gate, int gate_stride,
                                     const int* positions, const int* token_slot,
                                     const int* block_table, int tokens, int hq, int hkv, int d,
                                     int page_size, int num_pages, int max_pages, int slots,
@@ -135,7 +139,8 @@ extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache,
                                     int* fault, cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (d <= 0 || d % 16 != 0 || d > rl::kGenericWideD || hkv <= 0 || hq % hkv != 0 ||
-      page_size <= 0 || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || softcap < 0.0f || kv_planes < 1 || kv_planes > 2)
+      page_size <= 0 || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || softcap < 0.0f ||
+      out_stride < hq * d || (gate != nullptr && gate_stride < hq) || kv_planes < 1 || kv_planes > 2)
     return static_cast<int>(cudaErrorInvalidValue);
   const long long items = static_cast<long long>(tokens) * hq;
   const unsigned blocks =
@@ -145,7 +150,7 @@ extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache,
                                         : rl::attention_generic_kernel<scalar_t, rl::kGenericWideD>;
     kernel<<<blocks, rl::kGenericWarps * 32, 0, stream>>>(
         static_cast<const scalar_t*>(q), static_cast<const scalar_t*>(cache),
-        static_cast<scalar_t*>(out), positions, token_slot, block_table, tokens, hq, hkv, d,
+        static_cast<scalar_t*>(out), out_stride, static_cast<const scalar_t*>(gate), gate_stride, positions, token_slot, block_table, tokens, hq, hkv, d,
         page_size, num_pages, max_pages, slots, window, chunk, scale, softcap, sink, kv_planes, fault);
   });
   return rl::launch_status();

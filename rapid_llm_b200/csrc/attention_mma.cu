@@ -55,7 +55,7 @@ constexpr int kStagedPages = 1024;          // page ids of an item's key range k
 struct AttentionArgs {
   const bf16* q;            // [tokens, hq, D]
   const bf16* cache;        // [num_pages, 2, hkv, page_size, D]
-  bf16* out;                // [tokens, hq, D]
+  bf16* out;                // [tokens, hq, D], rows out_stride elements apart
   float* part_out;          // [tokens, hq, splits, D]   (splits > 1)
   float* part_lse;          // [tokens, hq, splits]      base-2 log-sum-exp
   const int* items;         // [n_items, 4]: entry, first packed row, split, unused
@@ -72,6 +72,9 @@ struct AttentionArgs {
   float scale;              // the plain scale (used with softcap)
   float softcap;            // 0 = scores are not squashed
   const float* sink;        // null = no sink
+  int out_stride;           // a multiple of 8
+  const bf16* gate;         // [tokens, hq] (rows gate_stride apart) or null: a head's output is multiplied by its sigmoid
+  int gate_stride;
   int kv_planes;            // 2; or 1 for a cache [num_pages, 1, hkv, page_size, D] whose rows are keys and values at once
                             // (the mma.sync tiles only)
 };
@@ -424,7 +427,8 @@ attention_mma_kernel(const AttentionArgs args) {
         inv = keys / (run_sum[i] * keys + exp2f(sink2 - top));
       }
       if (args.splits == 1) {
-        bf16* dst = args.out + row * kD + (lane & 3) * 2;
+        inv *= head_gate(args.gate, args.gate_stride, row_token[i], row_head[i]);
+        bf16* dst = args.out + static_cast<size_t>(row_token[i]) * args.out_stride + row_head[i] * kD + (lane & 3) * 2;
 #pragma unroll
         for (int nt = 0; nt < kD / 8; ++nt)
           *reinterpret_cast<__nv_bfloat162*>(dst + nt * 8) =
@@ -476,17 +480,17 @@ attention_mma_kernel(const AttentionArgs args) {
         value += weight * merge_o[(w * 16 + r) * kMergeStride + c];
       }
       float inv = total > 0.0f ? 1.0f / total : 0.0f;
-      const int token = p / group;
-      const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group +
-                         (p - token * group);
+      const int token = p / group, head = kv_head * group + (p - token * group);
+      const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + head;
       if (args.splits == 1 && args.sink != nullptr) {
-        const float sink2 = args.sink[kv_head * group + (p - token * group)] * 1.4426950408889634f;
+        const float sink2 = args.sink[head] * 1.4426950408889634f;
         const float top = fmaxf(m, sink2);
         const float keys = m == -INFINITY ? 0.0f : exp2f(m - top);
         inv = keys / (total * keys + exp2f(sink2 - top));
       }
       if (args.splits == 1) {
-        args.out[row * kD + c] = __float2bfloat16_rn(value * inv);
+        inv *= head_gate(args.gate, args.gate_stride, tok_begin + token, head);
+        args.out[static_cast<size_t>(tok_begin + token) * args.out_stride + head * kD + c] = __float2bfloat16_rn(value * inv);
       } else {
         args.part_out[(row * args.splits + split) * kD + c] = value * inv;
         if (c == 0)
@@ -499,8 +503,9 @@ attention_mma_kernel(const AttentionArgs args) {
 // out[row] = sum_s w_s part[row, s] / sum_s w_s with w_s = 2^(lse_s - max lse), splits in index
 // order; one warp per (token, head) row.
 __global__ void attention_merge_kernel(const float* __restrict__ part_out,
-                                       const float* __restrict__ part_lse, bf16* __restrict__ out,
-                                       long long rows, int splits, const float* __restrict__ sink, int hq) {
+                                       const float* __restrict__ part_lse, bf16* out,
+                                       long long rows, int splits, const float* __restrict__ sink, int hq,
+                                       int out_stride, const bf16* gate, int gate_stride) {
   pdl_trigger();
   pdl_wait();
   const long long row = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
@@ -513,7 +518,9 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_out,
   const float safe = m == -INFINITY ? 0.0f : m;
   float total = sink ? exp2f(sink2 - safe) : 0.0f;      // the sink counts once, whatever the number of parts
   for (int s = 0; s < splits; ++s) total += exp2f(lse[s] - safe);
-  const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+  const int token = static_cast<int>(row / hq), head = static_cast<int>(row - static_cast<long long>(token) * hq);
+  const float inv = (total > 0.0f ? 1.0f / total : 0.0f) * head_gate(gate, gate_stride, token, head);
+  bf16* dst = out + static_cast<size_t>(token) * out_stride + head * kD;
   for (int c = lane; c < kD; c += 32) {
     float value = 0.0f;
     for (int s = 0; s < splits; ++s) {
@@ -521,7 +528,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_out,
       if (lse[s] == -INFINITY) continue;
       value += exp2f(lse[s] - safe) * part_out[(row * splits + s) * kD + c];
     }
-    out[row * kD + c] = __float2bfloat16_rn(value * inv);
+    dst[c] = __float2bfloat16_rn(value * inv);
   }
 }
 
@@ -584,6 +591,7 @@ static int launch_prefill_tc(const AttentionArgs& a, int n_items, bool pdl, cuda
   t.entry_slot = a.entry_slot; t.block_table = a.block_table; t.hq = a.hq; t.hkv = a.hkv;
   t.page_size = a.page_size; t.num_pages = a.num_pages; t.max_pages = a.max_pages; t.slots = a.slots;
   t.window = a.window; t.chunk = a.chunk; t.scale_log2 = a.scale_log2; t.fault = a.fault;
+  t.out_stride = a.out_stride; t.gate = a.gate; t.gate_stride = a.gate_stride;
   t.softcap = a.softcap; t.sink = a.sink; t.cap_in = 0.0f; t.cap_out = 0.0f;
   if (a.softcap > 0.0f) {
     t.cap_in = 2.0f * 1.4426950408889634f * a.scale / a.softcap;
@@ -671,6 +679,7 @@ static int launch_decode_tc(const AttentionArgs& a, int n_items, int max_rows, b
   t.cu_seqlens = a.cu_seqlens; t.entry_start = a.entry_start; t.entry_slot = a.entry_slot;
   t.block_table = a.block_table; t.hq = a.hq; t.hkv = a.hkv; t.page_size = a.page_size;
   t.num_pages = a.num_pages; t.max_pages = a.max_pages; t.slots = a.slots; t.window = a.window;
+  t.out_stride = a.out_stride; t.gate = a.gate; t.gate_stride = a.gate_stride;
   t.chunk = a.chunk; t.sink = a.sink; t.splits = a.splits; t.cluster_merge = cluster_merge ? 1 : 0; t.scale_log2 = a.scale_log2; t.fault = a.fault;
   if (max_rows <= 0 || max_rows > kTcRows) max_rows = kTcRows;
   if (max_rows <= 1) return launch_decode_tc_rows<1>(map, t, n_items, pdl, stream, g_decode_tc_configured[0], rings);
@@ -737,7 +746,8 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
                      const int* entry_slot, const int* block_table, int tokens, int hq, int hkv,
                      int head_dim, int page_size, int num_pages, int max_pages, int slots,
                      int window, int chunk, int splits, float scale, int* fault, int pdl, int decode_kernel, int decode_rows,
-                     int chunk_rows, int decode_splits, float softcap, const float* sink, int kv_planes,
+                     int chunk_rows, int decode_splits, float softcap, const float* sink, int kv_planes, int out_stride,
+                     const void* gate, int gate_stride,
                      cudaStream_t stream) {
   if (tokens == 0 || (n_chunk_items == 0 && n_decode_items == 0)) return 0;
   if (softcap != 0.0f) {        // squashed scores: the tcgen05 chunk tiles and the mma.sync tiles take them
@@ -750,6 +760,9 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
   } else if (kv_planes != 2) {
     return static_cast<int>(cudaErrorInvalidValue);
   }
+  if (out_stride < hq * head_dim || out_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(out) & 15) ||
+      (gate != nullptr && gate_stride < hq))
+    return static_cast<int>(cudaErrorInvalidValue);
   if (head_dim != attn::kD || hkv <= 0 || hq % hkv != 0 || page_size <= 0 || window < 0 ||
       chunk < 0 || (window > 0 && chunk > 0) || splits < 1 || (splits > 1 && (part_out == nullptr || part_lse == nullptr)) ||
       hkv > 65535 || n_chunk_items > 65535 || n_decode_items > 65535)      // grid y dimensions
@@ -775,6 +788,7 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
   args.scale_log2 = scale * 1.4426950408889634f;
   args.fault = fault;
   args.scale = scale; args.softcap = softcap; args.sink = sink; args.kv_planes = kv_planes;
+  args.out_stride = out_stride; args.gate = static_cast<const attn::bf16*>(gate); args.gate_stride = gate_stride;
   int status = 0;
   bool merged_in_cluster = false;
   if (n_chunk_items > 0) {
@@ -808,7 +822,8 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
   if (splits > 1 && !merged_in_cluster) {
     const long long rows = static_cast<long long>(tokens) * hq;
     status = rl::launch_kernel(attn::attention_merge_kernel, dim3(static_cast<unsigned>((rows + 3) / 4)), dim3(128), 0,
-                               stream, pdl != 0, part_out, part_lse, static_cast<attn::bf16*>(out), rows, splits, sink, hq);
+                               stream, pdl != 0, part_out, part_lse, static_cast<attn::bf16*>(out), rows, splits, sink, hq,
+                               out_stride, static_cast<const attn::bf16*>(gate), gate_stride);
   }
   return status;
 }
@@ -900,7 +915,8 @@ int rl_attention_mma_static_scratch(const void* q, const void* cache, void* out,
   }
   return rl_attention_mma(q, cache, out, part_out, part_lse, chunk_items, n_chunk_items, decode_items,
                           n_decode_items, cu_seqlens, entry_start, entry_slot, block_table, tokens, hq, hkv,
-                          head_dim, page_size, num_pages, max_pages, slots, window, 0, splits, scale, fault, 0, 1, 0, 64, 0, 0.0f, nullptr, 2, stream);
+                          head_dim, page_size, num_pages, max_pages, slots, window, 0, splits, scale, fault, 0, 1, 0, 64, 0, 0.0f, nullptr, 2,
+                          hq * head_dim, nullptr, 0, stream);
 }
 
 }  // extern "C"

@@ -96,6 +96,9 @@ struct PrefillTcArgs {
   // cap_out * (1 - 2 / (1 + 2^(raw * cap_in))), cap_in = 2 log2(e) scale / softcap, cap_out = softcap log2(e).
   float softcap, cap_in, cap_out;
   const float* sink;
+  int out_stride;           // elements from a token's row of out to the next
+  const bf16* gate;         // [tokens, hq] or null: a head's output is multiplied by sigmoid(gate)
+  int gate_stride;
 };
 
 __device__ __forceinline__ float pf_fast_rcp(float x) {
@@ -466,7 +469,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const
     // the rows that exist are stored)
     if (ok && my_blocks > 0) ok = mbar_wait(smem_addr(&value_done[tile]), (my_blocks - 1) & 1, aborted, args.fault, 1 << (21 + tile));
     const bool all_ok = __all_sync(0xffffffffu, ok);
-    bf16* dst = args.out + (static_cast<size_t>(tok_begin + token) * args.hq + kv_head * group + (p - token * group)) * kPfD;
+    const int head = kv_head * group + (p - token * group);
+    bf16* dst = args.out + static_cast<size_t>(tok_begin + token) * args.out_stride + head * kPfD;
     if (all_ok && my_blocks > 0) {
       tc_fence_after();
       float even, odd;
@@ -474,10 +478,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const
       float row_sum = even + odd;
       if (args.sink != nullptr && valid) {
         // the sink's term against the same reference point as the keys' (an infinite one: it alone counts, the row is zero)
-        const float sink2 = args.sink[kv_head * group + (p - token * group)] * 1.4426950408889634f;
+        const float sink2 = args.sink[head] * 1.4426950408889634f;
         row_sum += fast_exp2(sink2 - (ref_max == -INFINITY ? 0.0f : ref_max));
       }
-      const float inv = row_sum > 0.0f ? 1.0f / row_sum : 0.0f;
+      float inv = row_sum > 0.0f ? 1.0f / row_sum : 0.0f;
+      if (valid) inv *= head_gate(args.gate, args.gate_stride, tok_begin + token, head);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         uint32_t raw[32];

@@ -110,6 +110,13 @@ __device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
   return window > 0 ? max(0, pos - window + 1) : 0;
 }
 
+// A gate of one number per token and head, applied to a head's output: sigmoid(gate[token * stride + head]), or 1
+// without a gate.
+template <typename T>
+__device__ __forceinline__ float head_gate(const T* gate, int stride, int token, int head) {
+  return gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-to_float(gate[static_cast<size_t>(token) * stride + head])));
+}
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // ---- programmatic dependent launch -------------------------------------------------------

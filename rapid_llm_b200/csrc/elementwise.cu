@@ -341,13 +341,12 @@ __global__ void layernorm_kernel(const T* __restrict__ x, float* __restrict__ re
   }
 }
 
-// ------------------------------------------------------------ a sigmoid gate, entry by entry or one number a head
-// out[t, c] = rows[t, c] * sigmoid(gate[t, c / per]), float32 arithmetic, one rounding; `per` 1: a number an entry,
-// or the head size: a number a head.  `gate` and `out` may be views of some columns of wider rows (their strides), and
-// of the same rows (not of the same columns).  kVector: eight entries (16 bytes of bfloat16) a thread and step.
+// ------------------------------------------------------------ a sigmoid gate, entry by entry
+// out[t, c] = rows[t, c] * sigmoid(gate[t, c]), float32 arithmetic, one rounding; `gate` and `out` may be views of some
+// columns of wider rows (their strides), and of the same rows (not of the same columns).  kVector: eight entries (16 bytes of bfloat16) a thread and step.
 template <typename T, bool kVector>
 __global__ void sigmoid_gate_kernel(const T* __restrict__ rows, const T* gate, int gate_stride,
-                                    T* out, int out_stride, int tokens, int width, int per) {
+                                    T* out, int out_stride, int tokens, int width) {
   pdl_trigger();
   pdl_wait();
   constexpr int kStep = kVector ? 8 : 1;
@@ -360,18 +359,12 @@ __global__ void sigmoid_gate_kernel(const T* __restrict__ rows, const T* gate, i
     if constexpr (kVector) {
       float v[8], g[8];
       load8(rows + t * width + c, v);
-      if (per > 1) {       // a head's size is a multiple of eight here: the eight entries share their number
-        const float factor = 1.0f / (1.0f + expf(-to_float(gate[t * gate_stride + c / per])));
+      load8(gate + t * gate_stride + c, g);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) v[i] *= factor;
-      } else {
-        load8(gate + t * gate_stride + c, g);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) v[i] = v[i] / (1.0f + expf(-g[i]));
-      }
+      for (int i = 0; i < 8; ++i) v[i] = v[i] / (1.0f + expf(-g[i]));
       store8(out + t * out_stride + c, v);
     } else {
-      const float g = to_float(gate[t * gate_stride + c / per]);
+      const float g = to_float(gate[t * gate_stride + c]);
       out[t * out_stride + c] = from_float<T>(to_float(rows[t * width + c]) / (1.0f + expf(-g)));
     }
   }
@@ -602,12 +595,11 @@ int rl_layernorm(int dtype, const void* x, float* residual, const float* weight,
 }
 
 int rl_sigmoid_gate(int dtype, const void* rows, const void* gate, int gate_stride, void* out, int out_stride, int tokens,
-                    int width, int per, int pdl, cudaStream_t stream) {
+                    int width, int pdl, cudaStream_t stream) {
   if (tokens == 0 || width == 0) return 0;
-  if (width < 0 || per < 1 || width % per != 0 || gate_stride < width / per || out_stride < width)
-    return static_cast<int>(cudaErrorInvalidValue);
-  const bool vector = width % 8 == 0 && out_stride % 8 == 0 && rl::aligned16(rows) && rl::aligned16(out) &&
-                      (per > 1 ? per % 8 == 0 : gate_stride % 8 == 0 && rl::aligned16(gate));
+  if (width < 0 || gate_stride < width || out_stride < width) return static_cast<int>(cudaErrorInvalidValue);
+  const bool vector = width % 8 == 0 && gate_stride % 8 == 0 && out_stride % 8 == 0 && rl::aligned16(rows) &&
+                      rl::aligned16(gate) && rl::aligned16(out);
   const size_t total = static_cast<size_t>(tokens) * (vector ? width / 8 : width);
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
@@ -615,7 +607,7 @@ int rl_sigmoid_gate(int dtype, const void* rows, const void* gate, int gate_stri
     auto kernel = vector ? rl::sigmoid_gate_kernel<scalar_t, true> : rl::sigmoid_gate_kernel<scalar_t, false>;
     return rl::launch_kernel(kernel, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream, pdl != 0,
                              static_cast<const scalar_t*>(rows), static_cast<const scalar_t*>(gate), gate_stride,
-                             static_cast<scalar_t*>(out), out_stride, tokens, width, per);
+                             static_cast<scalar_t*>(out), out_stride, tokens, width);
   });
   return 0;
 }

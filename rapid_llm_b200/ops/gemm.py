@@ -30,6 +30,7 @@ weight stream gains over kernels chained by programmatic dependent launch.
 
 from __future__ import annotations
 
+import weakref
 from dataclasses import dataclass
 from typing import Any
 
@@ -126,15 +127,18 @@ def use_tensor_core_kernel(x: torch.Tensor, weight: torch.Tensor) -> bool:
     return x.shape[0] <= TENSOR_CORE_MAX_TOKENS
 
 
-_BIAS_IN_DTYPE: dict[tuple[int, torch.dtype], torch.Tensor] = {}
+_BIAS_IN_DTYPE: dict[tuple[int, torch.dtype], tuple] = {}
 
 
 def _bias_as(bias: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
-    """The float32 bias in the product's dtype for the library call (made once per vector)."""
-    key = (bias.data_ptr(), dtype)
-    if key not in _BIAS_IN_DTYPE:
-        _BIAS_IN_DTYPE[key] = bias.to(dtype)
-    return _BIAS_IN_DTYPE[key]
+    """The float32 bias in the product's dtype for the library call, made once per vector and kept as long as the vector
+    lives (an address alone would name the vector that was there before)."""
+    key = (id(bias), dtype)
+    kept = _BIAS_IN_DTYPE.get(key)
+    if kept is None or kept[0]() is not bias or kept[1] != bias._version:
+        owner = weakref.ref(bias, lambda _: _BIAS_IN_DTYPE.pop(key, None))
+        kept = _BIAS_IN_DTYPE[key] = (owner, bias._version, bias.to(dtype))
+    return kept[2]
 
 
 def linear(x, weight: torch.Tensor, out: torch.Tensor, fault: torch.Tensor | None = None, *,

@@ -124,7 +124,7 @@ def core() -> ctypes.CDLL:
             c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
         ]
-        lib.rl_sigmoid_gate.argtypes = [c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
+        lib.rl_sigmoid_gate.argtypes = [c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.rl_relu_squared.argtypes = [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.rl_silu_mul.argtypes = [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
         lib.rl_clamped_glu.argtypes = [c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p]
@@ -140,7 +140,7 @@ def core() -> ctypes.CDLL:
             c_float, c_int, c_void_p, c_int, c_void_p,
         ]
         lib.rl_attention_generic.argtypes = [
-            c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+            c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p,
         ]
         lib.rl_embedding_sum.argtypes = [
@@ -370,16 +370,14 @@ def row_norm_rope_write(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: in
 
 
 def sigmoid_gate(rows: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """``out = rows * sigmoid(gate)`` (float32 arithmetic): entry by entry, or, with a ``gate [T, heads]``, one number
-    for all entries of a head.  ``gate`` and ``out`` may be views of some columns of wider rows."""
+    """``out = rows * sigmoid(gate)`` entry by entry (float32 arithmetic); ``gate`` and ``out`` may be views of some
+    columns of wider rows."""
     _need_cuda(rows, gate, out)
     _contig("rows", rows)
-    if (gate.shape[0] != rows.shape[0] or rows.shape[1] % gate.shape[1] or out.shape != rows.shape
-            or gate.dtype != rows.dtype or out.dtype != rows.dtype):
+    if gate.shape != rows.shape or out.shape != rows.shape or gate.dtype != rows.dtype or out.dtype != rows.dtype:
         raise KernelError("sigmoid_gate: shapes or dtypes do not agree")
     _check(core().rl_sigmoid_gate(dtype_tag(rows.dtype), _ptr(rows), _ptr(gate), _row_stride("gate", gate), _ptr(out),
-                                  _row_stride("out", out), rows.shape[0], rows.shape[1], rows.shape[1] // gate.shape[1],
-                                  int(PDL), _stream()), "sigmoid_gate")
+                                  _row_stride("out", out), rows.shape[0], rows.shape[1], int(PDL), _stream()), "sigmoid_gate")
     return out
 
 
@@ -532,16 +530,18 @@ def attention_generic(
     softcap: float = 0.0,
     sink: torch.Tensor | None = None,
     chunk: int = 0,
+    gate: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """Causal attention of every token of the step over its request's cached keys: all of them, the last ``window``
     positions, or (``chunk`` > 0) those of the position's own chunk, counted from position 0.  ``softcap`` > 0 squashes the
     scaled scores to ``softcap * tanh(s / softcap)``; ``sink`` (float32 ``[heads]``) adds ``exp(sink[h])`` to every
-    row's denominator."""
-    _need_cuda(q, cache, out, positions, token_slot, block_table, fault, sink)
+    row's denominator; ``gate`` (``[T, heads]``) multiplies a head's output by its sigmoid.  ``out`` (rows) and ``gate``
+    may be views of some columns of wider rows."""
+    _need_cuda(q, cache, out, positions, token_slot, block_table, fault, sink, gate)
     _expect("sink", sink, torch.float32), _contig("sink", sink)
     if sink is not None and sink.numel() != num_heads:
         raise KernelError("attention: one sink per head")
-    _contig("q", q), _contig("cache", cache), _contig("out", out), _contig("block_table", block_table)
+    _contig("q", q), _contig("cache", cache), _contig("block_table", block_table)
     for name, tensor in (("positions", positions), ("token_slot", token_slot), ("block_table", block_table)):
         _expect(name, tensor, torch.int32)
     tokens = positions.numel()
@@ -551,11 +551,12 @@ def attention_generic(
         raise KernelError("attention: q, cache and out must share a dtype")
     if cache.dim() != 5 or cache.shape[1] not in (1, 2) or cache.shape[2] != num_kv_heads or cache.shape[4] != head_dim:
         raise KernelError("attention: cache must be [pages, 2 (or 1: values are the keys' rows), kv_heads, page_size, head_dim]")
+    out_stride, gate_stride = _attention_out(out, gate, tokens, num_heads, head_dim)
     if head_dim % 16 or head_dim > 640:
         raise KernelError(f"attention: head_dim {head_dim} must be a multiple of 16 up to 640")
     _check(
         core().rl_attention_generic(
-            dtype_tag(q.dtype), _ptr(q), _ptr(cache), _ptr(out), _ptr(positions), _ptr(token_slot),
+            dtype_tag(q.dtype), _ptr(q), _ptr(cache), _ptr(out), out_stride, _ptr(gate), gate_stride, _ptr(positions), _ptr(token_slot),
             _ptr(block_table), tokens, num_heads, num_kv_heads, head_dim, cache.shape[3],
             cache.shape[0], block_table.shape[1], block_table.shape[0], int(window), int(chunk), float(scale),
             float(softcap), _ptr(sink), int(cache.shape[1]), _ptr(fault), _stream(),
@@ -563,6 +564,20 @@ def attention_generic(
         f"attention_generic(head_dim={head_dim})",
     )
     return out
+
+
+def _attention_out(out: torch.Tensor, gate: torch.Tensor | None, tokens: int, num_heads: int, head_dim: int) -> tuple[int, int]:
+    """Row strides of attention's ``out`` and ``gate``, their shapes checked."""
+    if out.dim() == 2 and out.shape == (tokens, num_heads * head_dim):
+        out_stride = _row_stride("out", out)
+    else:
+        _contig("out", out)
+        out_stride = num_heads * head_dim
+    if gate is None:
+        return out_stride, 0
+    if gate.shape != (tokens, num_heads) or gate.dtype != out.dtype:
+        raise KernelError("attention: the gate must be [tokens, heads] of the output's dtype")
+    return out_stride, _row_stride("gate", gate)
 
 
 _ATTENTION_LIBS: dict[int, ctypes.CDLL] = {}
@@ -590,7 +605,8 @@ def attention_lib(head_dim: int) -> ctypes.CDLL:
         lib.rl_attention_mma.argtypes = [
             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
+            c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int,
+            c_int, c_void_p, c_int, c_void_p,
         ]
         lib.rl_attention_mma.restype = c_int
         lib.rl_attention_decode_max_clusters.argtypes = [c_int]
@@ -648,6 +664,7 @@ def attention_mma(
     softcap: float = 0.0,
     sink: torch.Tensor | None = None,
     chunk: int = 0,
+    gate: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """bfloat16 paged causal attention over work items the host cut the step into.
 
@@ -668,15 +685,18 @@ def attention_mma(
     ``softcap`` > 0 squashes the scaled scores to ``softcap * tanh(s / softcap)``; ``sink`` (float32 ``[heads]``)
     adds ``exp(sink[h])`` to every row's denominator, once.  All tiles take a sink; with squashed scores the decode
     tiles run on mma.sync (and have no split count of their own).  A position sees all keys up to its own, or the last
-    ``window`` of them, or (``chunk`` > 0) those of its own chunk, chunks being counted from position 0.
+    ``window`` of them, or (``chunk`` > 0) those of its own chunk, chunks being counted from position 0.  ``gate``
+    (``[T, heads]``) multiplies a head's output by its sigmoid.  ``out`` and ``gate`` may be views of some columns of
+    wider rows.
     """
     _need_cuda(q, cache, out, chunk_items, decode_items, part_out, part_lse, cu_seqlens, entry_start,
-               entry_slot, block_table, fault, sink)
+               entry_slot, block_table, fault, sink, gate)
     _expect("sink", sink, torch.float32), _contig("sink", sink)
     if sink is not None and sink.numel() != num_heads:
         raise KernelError("attention: one sink per head")
     for name, tensor in (("q", q), ("cache", cache), ("out", out)):
-        _expect(name, tensor, torch.bfloat16), _contig(name, tensor)
+        _expect(name, tensor, torch.bfloat16)
+    _contig("q", q), _contig("cache", cache)
     for name, tensor in (("chunk_items", chunk_items), ("decode_items", decode_items), ("cu_seqlens", cu_seqlens),
                          ("entry_start", entry_start), ("entry_slot", entry_slot), ("block_table", block_table)):
         _expect(name, tensor, torch.int32), _contig(name, tensor)
@@ -689,6 +709,7 @@ def attention_mma(
         raise KernelError("attention: cache must be [pages, 2 (or 1: values are the keys' rows), kv_heads, page_size, head_dim]")
     if num_heads % num_kv_heads:
         raise KernelError("attention: heads must be a multiple of kv heads")
+    out_stride, gate_stride = _attention_out(out, gate, tokens, num_heads, head_dim)
     n_chunk = 0 if chunk_items is None else chunk_items.shape[0]
     n_decode = 0 if decode_items is None else decode_items.shape[0]
     if splits > 1:
@@ -702,7 +723,7 @@ def attention_mma(
             _ptr(block_table), tokens, num_heads, num_kv_heads, head_dim, cache.shape[3], cache.shape[0],
             block_table.shape[1], block_table.shape[0], int(window), int(chunk), int(splits), float(scale),
             _ptr(fault), int(PDL), {"auto": 0, "mma": 1, "deep": 2, "shallow": 3}[decode_kernel], int(decode_rows), int(chunk_rows),
-            int(decode_splits), float(softcap), _ptr(sink), int(cache.shape[1]), _stream(),
+            int(decode_splits), float(softcap), _ptr(sink), int(cache.shape[1]), out_stride, _ptr(gate), gate_stride, _stream(),
         ),
         f"attention_mma(head_dim={head_dim})",
     )

@@ -463,21 +463,19 @@ class GQAAttention(Mixer):
         rows = x.shape[0]
         qkv = batch.workspace.get("attn_qkv", rows, self.qkv.shape[0], x.dtype)
         gemm.linear(x, self.qkv, qkv, batch.fault, bias=self.qkv_bias, defer=batch.defer_products)
-        attended = self._attended(qkv, batch, cache)
-        if self.gate:
-            if self.gate_rides:
-                gate = qkv[:, self.qkv_rows : self.qkv_rows + self.gate_width]          # the first product brought it along
-            else:
-                gate = batch.workspace.get("attn_gate", rows, self.gate_width, x.dtype)
-                gemm.linear(x, self.g, gate, batch.fault)
-            gated = batch.workspace.get("attn_gated", rows, self.hq * self.d, x.dtype)
-            attended = kernels.sigmoid_gate(attended, gate, gated)
+        gate = None
+        if self.gate_rides:
+            gate = qkv[:, self.qkv_rows : self.qkv_rows + self.gate_width]          # the first product brought it along
+        elif self.gate:
+            gate = batch.workspace.get("attn_gate", rows, self.gate_width, x.dtype)
+            gemm.linear(x, self.g, gate, batch.fault)
+        attended = self._attended(qkv, gate, batch.workspace.get("attn_heads", rows, self.hq * self.d, x.dtype), batch, cache)
         out = batch.workspace.get("attn_proj", rows, self.hidden, x.dtype)
         return gemm.linear(attended, self.o, out, batch.fault, then_norm=then_norm, bias=self.o_bias, defer=batch.defer_products)
 
-    def _attended(self, qkv, batch, cache) -> torch.Tensor:
-        """From the first product's result to the heads side by side, before the gate: norms, rotation, the cache's
-        store and attention."""
+    def _attended(self, qkv, gate, out, batch, cache) -> torch.Tensor:
+        """From the first product's result to the gated heads side by side in ``out``: norms, rotation, the cache's store,
+        attention (whose last step a gate of one number a head is) and a gate entry by entry."""
         if cache.group is None or cache.pages is None:
             raise ValueError("attention needs a cache group; the engine did not give this layer one")
         if cache.writes == self.shares_cache:
@@ -496,14 +494,17 @@ class GQAAttention(Mixer):
                 page_size=group.page_size, neighbours=self.neighbours, values_are_keys=self.keys_are_values)
         else:
             self._norm_rope_write(qkv, q, batch, cache, group)
+        if self.gate != "sigmoid":
+            self.attend(q, cache.pages, out, batch, group, gate)
+            return out
         attended = batch.workspace.get("attn_out", rows, self.hq * self.d, qkv.dtype)
         self.attend(q, cache.pages, attended, batch, group)
-        return attended
+        return kernels.sigmoid_gate(attended, gate, out)
 
     # -- in an arrangement that stacks its sublayers' products ------------------- #
     @property
     def stacks(self) -> bool:
-        return self.gate_rides and not self.float_prelude
+        return self.row_norm and not self.float_prelude
 
     @property
     def first_rows(self) -> int:
@@ -516,15 +517,16 @@ class GQAAttention(Mixer):
     def adopt(self, first, first_bias, last) -> None:
         """Keep the weights of the first and the last product in the arrangement's matrices (views) from here on."""
         self.qkv, self.o = first, last
-        self.g = self._riding_gate()
+        if self.gate:
+            self.g = self._riding_gate()
         if self.qkv_bias is not None:
             self.qkv_bias = first_bias
 
     def middle(self, wide, batch, cache) -> None:
         """``wide [T, first_rows]``, the first product's result (a view of some columns of wider rows), in; the last
         product's input in its first ``last_columns`` columns, out: the gated heads take the queries' place."""
-        attended = self._attended(wide, batch, cache)
-        kernels.sigmoid_gate(attended, wide[:, self.qkv_rows : self.qkv_rows + self.gate_width], wide[:, : self.last_columns])
+        gate = wide[:, self.qkv_rows : self.qkv_rows + self.gate_width] if self.gate else None
+        self._attended(wide, gate, wide[:, : self.last_columns], batch, cache)
 
     def _float_prelude(self, qkv, q, batch, cache, group) -> None:
         """Projection -> short convolution (float32, the slot's tail before the step's rows) -> rotation ->
@@ -564,7 +566,7 @@ class GQAAttention(Mixer):
             page_size=group.page_size, norm_size=self.qk_dim,
         )
 
-    def attend(self, q, pages, out, batch, group) -> None:
+    def attend(self, q, pages, out, batch, group, gate=None) -> None:
         if q.dtype == torch.bfloat16:
             plan = batch.extras[self._items.key]
             splits = plan["splits"]
@@ -582,6 +584,7 @@ class GQAAttention(Mixer):
                 window=self.window, scale=self.scale, fault=batch.fault, decode_rows=plan.get("decode_rows", 0),
                 chunk_rows=plan.get("chunk_rows", kernels.CHUNK_TILE_ROWS),
                 decode_splits=plan.get("decode_splits", 0), softcap=self.softcap, sink=self.sink, chunk=self.chunk,
+                gate=gate,
             )
             return
         kernels.attention_generic(
@@ -589,4 +592,5 @@ class GQAAttention(Mixer):
             positions=batch.positions, token_slot=batch.token_slot, block_table=group.block_table,
             num_heads=self.hq, num_kv_heads=self.hkv, head_dim=self.d,
             window=self.window, scale=self.scale, fault=batch.fault, softcap=self.softcap, sink=self.sink, chunk=self.chunk,
+            gate=gate,
         )
