@@ -12,7 +12,7 @@ of 512 positions, a feed-forward of ``4 W``.  Zupupel, Mezadra and Qwen3 beside 
 (Qwen3's gated feed-forward has ``8 W / 3``, the same number of weights).  Prefill is one 2,048-token step (best of
 three, CUDA events around the step function); decode is batch 8 behind 1,024-token prompts, replayed from the captured
 graph (median of 32 steps).  Kernels are timed alone with CUDA events, L2 flushed between runs (a write of 256 MB), on one
-2,048-token prompt and on 64 (products also on 8) single tokens behind 1,024 cached ones; ``frac`` is (bytes the kernel
+2,048-token prompt and on 64 (products also on 8) single tokens behind 1,535 cached ones (the last of their chunk); ``frac`` is (bytes the kernel
 must move) / time / measured copy bandwidth, ``tflops`` the products' arithmetic over the same time.
 """
 
@@ -77,7 +77,7 @@ def kernel_figures(width: int, hbm_gbs: float) -> dict:
     f32 = lambda *shape: torch.randn(*shape, device=device)                        # noqa: E731
     fault = torch.zeros(1, dtype=torch.int32, device=device)
     workspace = SimpleNamespace(get=lambda name, rows, cols, dtype, min_rows=None: torch.empty(rows, cols, dtype=dtype, device=device))
-    page, context = 16, 1024
+    page, context = 16, 1535       # the single tokens are the last of a chunk: they see as many keys as the window lets them
     mix_rows = (heads + kv_heads) * d + -(-heads // 8) * 8
     first, last = bf(ff + mix_rows, width) / width ** 0.5, bf(width, ff + heads * d) / width ** 0.5
     first_bias, out_bias = f32(ff + mix_rows), f32(width)

@@ -133,11 +133,10 @@ class AttentionItems(StepPlanner):
         lengths = np.asarray(shape.lengths, dtype=np.int64)
         starts = np.asarray(shape.starts, dtype=np.int64)
         rows = lengths * self.group
-        # keys before the step's first and last position of an entry, as far as its rows walk them
-        seen_first, seen_last = starts, starts + lengths
+        # the most keys a tile of an entry walks
+        seen_last = starts + lengths
         if self.chunk:
-            seen_first = starts % self.chunk
-            seen_last = np.minimum(seen_first + lengths, self.chunk + lengths - 1)
+            seen_last = np.minimum(starts % self.chunk + lengths, self.chunk + lengths - 1)
         is_decode = (lengths == 1) | (rows <= kernels.DECODE_TILE_ROWS)
         tensor_core = self.tensor_core and kernels.attention_tc_takes(self.head_dim, shape.page_size)
         for chunk_rows in ((kernels.CHUNK_TILE_ROWS_TC, kernels.CHUNK_TILE_ROWS) if tensor_core else (kernels.CHUNK_TILE_ROWS,)):
@@ -188,7 +187,10 @@ class AttentionItems(StepPlanner):
         row0 = tile_index * np.repeat(tile_rows, tiles)
         decode_tile = np.repeat(is_decode, tiles)
         # keys a tile has to walk: the tiles with the most go first, so that the last wave is short
-        keys = np.repeat(seen_first, tiles) + (row0 + np.repeat(tile_rows, tiles)) // self.group
+        keys = np.repeat(starts, tiles) + (row0 + np.repeat(tile_rows, tiles)) // self.group
+        if self.chunk:
+            first_position = np.repeat(starts, tiles) + row0 // self.group
+            keys = keys - (first_position - first_position % self.chunk)
 
         def items(mask: np.ndarray, ranges: int) -> np.ndarray:
             order = np.flatnonzero(mask)

@@ -43,13 +43,13 @@ def frequencies(dims: int, base: float, scaling: dict | None) -> list[float]:
 def rotate_neighbours(rows: torch.Tensor, dims: int, freq: list[float]) -> torch.Tensor:
     """Rotate the first ``dims`` entries of ``rows [T, heads, n]``: entries ``2i`` and ``2i + 1`` of the row at position
     ``p`` turn by ``p * freq[i]``."""
+    if dims == 0:
+        return rows
+    angle = torch.arange(rows.shape[0], dtype=F64)[:, None] * torch.tensor(freq, dtype=F64)[None, :]
+    cos, sin = torch.cos(angle)[:, None, :], torch.sin(angle)[:, None, :]
+    u, v = rows[..., 0:dims:2], rows[..., 1:dims:2]
     out = rows.clone()
-    for p in range(rows.shape[0]):
-        for i in range(dims // 2):
-            cos, sin = math.cos(p * freq[i]), math.sin(p * freq[i])
-            u, v = rows[p, :, 2 * i], rows[p, :, 2 * i + 1]
-            out[p, :, 2 * i] = u * cos - v * sin
-            out[p, :, 2 * i + 1] = v * cos + u * sin
+    out[..., 0:dims:2], out[..., 1:dims:2] = u * cos - v * sin, v * cos + u * sin
     return out
 
 
