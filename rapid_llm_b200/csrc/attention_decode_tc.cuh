@@ -91,8 +91,9 @@ __device__ __forceinline__ float warp_max_redux(float v) {
 }
 
 // kRows: how many of the 16 columns of the products carry query rows (a power of two); the
-// per-row work of the softmax threads is unrolled over exactly these.
-template <int kRows, int kTcStages>
+// per-row work of the softmax threads is unrolled over exactly these.  kDressed: the row's last step knows a sink, a
+// gate and an output whose rows are some columns of wider ones (the plain form keeps its registers and its short tail).
+template <int kRows, int kTcStages, bool kDressed>
 __global__ void __launch_bounds__(kTcThreads, kTcStages == 1 ? 2 : 1)
 attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const DecodeTcArgs args) {
   static_assert(kRows >= 1 && kRows <= kTcRows && (kRows & (kRows - 1)) == 0, "rows: a power of two up to 16");
@@ -479,17 +480,17 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
       const float lse = total > 0.0f ? m + log2f(total) : -INFINITY;
       const int p = row0 + n, token = p / group, head = kv_head * group + (p - token * group);
       const size_t row = static_cast<size_t>(tok_begin + token) * args.hq + head;
-      if (args.sink != nullptr && args.splits == 1) {
+      if (kDressed && args.sink != nullptr && args.splits == 1) {
         // an unsplit row's denominator takes the sink here; a split one's where its parts meet
         const float sink2 = args.sink[head] * 1.4426950408889634f;
         const float top = fmaxf(m, sink2);
         const float keys = m == -INFINITY ? 0.0f : fast_exp2(m - top);
         inv = keys / (total * keys + fast_exp2(sink2 - top));
       }
-      if (args.splits == 1) inv *= head_gate(args.gate, args.gate_stride, tok_begin + token, head);
+      if (kDressed && args.splits == 1) inv *= head_gate(args.gate, args.gate_stride, tok_begin + token, head);
       const float merged = value * inv;
       if (args.splits == 1) {
-        args.out[static_cast<size_t>(tok_begin + token) * args.out_stride + head * kTcD + t] = __float2bfloat16_rn(merged);
+        args.out[(kDressed ? static_cast<size_t>(tok_begin + token) * args.out_stride + head * kTcD : row * kTcD) + t] = __float2bfloat16_rn(merged);
       } else if (args.cluster_merge) {
         split_out[n * 128 + t] = merged;
         if (t == 0) split_lse[n] = lse;
@@ -536,8 +537,8 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
           }
         }
         const int p = row0 + n, token = p / group, head = kv_head * group + (p - token * group);
-        const float sink2 = args.sink != nullptr ? args.sink[head] * 1.4426950408889634f : -INFINITY;
-        const float factor = head_gate(args.gate, args.gate_stride, tok_begin + token, head);
+        const float sink2 = kDressed && args.sink != nullptr ? args.sink[head] * 1.4426950408889634f : -INFINITY;
+        const float factor = kDressed ? head_gate(args.gate, args.gate_stride, tok_begin + token, head) : 1.0f;
         float m = sink2;
 #pragma unroll
         for (int r = 0; r < 8; ++r) m = fmaxf(m, lse_of[r]);
@@ -546,7 +547,7 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
           for (int r = 8; r < kTcMaxClusterSplits; ++r) m = fmaxf(m, lse_of[r]);
         }
         const float safe = m == -INFINITY ? 0.0f : m;
-        float total = args.sink != nullptr ? fast_exp2(sink2 - safe) : 0.0f, value = 0.0f;
+        float total = kDressed && args.sink != nullptr ? fast_exp2(sink2 - safe) : 0.0f, value = 0.0f;
 #pragma unroll
         for (int r = 0; r < 8; ++r) {
           if (r < args.splits) {
@@ -565,8 +566,9 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
             }
           }
         }
-        args.out[static_cast<size_t>(tok_begin + token) * args.out_stride + head * kTcD + t] =
-            __float2bfloat16_rn(total > 0.0f ? value / total * factor : 0.0f);
+        const size_t at = kDressed ? static_cast<size_t>(tok_begin + token) * args.out_stride + head * kTcD
+                                   : (static_cast<size_t>(tok_begin + token) * args.hq + head) * kTcD;
+        args.out[at + t] = __float2bfloat16_rn(total > 0.0f ? value / total * factor : 0.0f);
       }
     }
     __syncwarp();

@@ -601,7 +601,7 @@ static int launch_prefill_tc(const AttentionArgs& a, int n_items, bool pdl, cuda
                        map, t);
 }
 
-static bool g_decode_tc_configured[5][2] = {};   // per row-count and ring-depth instantiation; file-local on purpose
+static bool g_decode_tc_configured[5][2][2] = {};   // per row-count, ring-depth and dressed instantiation; file-local on purpose
 
 static int decode_tc_sm_count() {
   int device = 0, sms = 0;
@@ -611,10 +611,10 @@ static int decode_tc_sm_count() {
   return sms;
 }
 
-template <int kRows, int kStages>
-static int launch_decode_tc_stages(const CUtensorMap& map, const DecodeTcArgs& t, int n_items, bool pdl,
+template <int kRows, int kStages, bool kDressed>
+static int launch_decode_tc_as(const CUtensorMap& map, const DecodeTcArgs& t, int n_items, bool pdl,
                                    cudaStream_t stream, bool* configured) {
-  auto kernel = attention_decode_tc_kernel<kRows, kStages>;
+  auto kernel = attention_decode_tc_kernel<kRows, kStages, kDressed>;
   constexpr int kTcSmemBytes = tc_smem_bytes(kStages);
   if (!*configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmemBytes);
@@ -652,17 +652,25 @@ static int launch_decode_tc_stages(const CUtensorMap& map, const DecodeTcArgs& t
   return static_cast<int>(cudaLaunchKernelEx(&config, kernel, map, t));
 }
 
+template <int kRows, int kStages>
+static int launch_decode_tc_stages(const CUtensorMap& map, const DecodeTcArgs& t, int n_items, bool pdl,
+                                   cudaStream_t stream, bool* configured) {
+  const bool dressed = t.sink != nullptr || t.gate != nullptr || t.out_stride != t.hq * kTcD;
+  if (dressed) return launch_decode_tc_as<kRows, kStages, true>(map, t, n_items, pdl, stream, configured + 1);
+  return launch_decode_tc_as<kRows, kStages, false>(map, t, n_items, pdl, stream, configured);
+}
+
 // More CTAs than multiprocessors, each by itself (no cluster): two shallow CTAs per multiprocessor, so that one
 // streams while the other starts.  Decided by the number of items alone: a captured decode graph replays the same
 // choice at every context length.
 // `rings`: 0 = decide here, 2 = deep, 3 = shallow (for measurements).
 template <int kRows>
 static int launch_decode_tc_rows(const CUtensorMap& map, const DecodeTcArgs& t, int n_items, bool pdl,
-                                 cudaStream_t stream, bool* configured, int rings) {
+                                 cudaStream_t stream, bool (*configured)[2], int rings) {
   const bool shallow = rings == 3 || (rings != 2 && !t.cluster_merge &&
                                       static_cast<long long>(n_items) * t.hkv > decode_tc_sm_count());
-  if (shallow) return launch_decode_tc_stages<kRows, 1>(map, t, n_items, pdl, stream, configured + 1);
-  return launch_decode_tc_stages<kRows, kTcMaxStages>(map, t, n_items, pdl, stream, configured);
+  if (shallow) return launch_decode_tc_stages<kRows, 1>(map, t, n_items, pdl, stream, configured[1]);
+  return launch_decode_tc_stages<kRows, kTcMaxStages>(map, t, n_items, pdl, stream, configured[0]);
 }
 
 // cluster_merge: the `splits` items of a tile are consecutive in the grid and launched as one
@@ -719,7 +727,7 @@ int rl_attention_decode_rows() { return 16; }
 // the number of multiprocessors over the size; the host's planner asks once per size.
 int rl_attention_decode_max_clusters(int cluster_size) {
   if (attn::kD != attn::kTcD || cluster_size < 1 || cluster_size > attn::kTcMaxClusterSplits) return -static_cast<int>(cudaErrorInvalidValue);
-  auto kernel = attn::attention_decode_tc_kernel<4, attn::kTcMaxStages>;
+  auto kernel = attn::attention_decode_tc_kernel<4, attn::kTcMaxStages, false>;
   constexpr int kBytes = attn::tc_smem_bytes(attn::kTcMaxStages);
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);

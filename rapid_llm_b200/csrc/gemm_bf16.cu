@@ -132,7 +132,8 @@ struct GemmShape {
 
 // grid = (k_split, tile CTAs); with k_split > 1 the x dimension is one cluster and every CTA
 // has exactly one tile; otherwise a CTA walks the tiles blockIdx.y, blockIdx.y + gridDim.y, ...
-template <bool kSwiglu, int BN>
+// kRelu2: the first relu2_columns columns of a plain product take the square of relu.
+template <bool kSwiglu, int BN, bool kRelu2>
 __global__ void __launch_bounds__(kGemmThreads)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                  const GemmArgs args) {
@@ -347,7 +348,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gated_unit(v[j], (scaled ? u[j] * row_scale[c + j] : u[j]) + bias_up, args.glu_limit, args.glu_alpha);
           }
-          if (!kSwiglu && n < args.relu2_columns) {
+          if (kRelu2 && n < args.relu2_columns) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = relu_squared(v[j]);
           }
@@ -442,7 +443,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
         for (int r = 0; r < 4; ++r) {
           const float g = gate[r] * scale + bias_gate[r], u = up[r] * scale + bias_up[r];
           result[r] = kSwiglu ? gated_unit(g, u, args.glu_limit, args.glu_alpha) : g;
-          if (!kSwiglu && n + r < args.relu2_columns) result[r] = relu_squared(result[r]);
+        }
+        if (kRelu2 && n < args.relu2_columns) {
+#pragma unroll
+          for (int r = 0; r < 4; ++r)
+            if (n + r < args.relu2_columns) result[r] = relu_squared(result[r]);
         }
         if (norm_follows) {
           float before[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -508,14 +513,15 @@ static int sm_count() {
   return sms;
 }
 
-static bool g_gemm_configured[2][9] = {};   // [swiglu][BN / 32]; file-local on purpose
+static bool g_gemm_configured[3][9] = {};   // [plain, swiglu, squared columns][BN / 32]; file-local on purpose
 
-template <bool kSwiglu, int BN>
+template <bool kSwiglu, int BN, bool kRelu2>
 static int launch_gemm(const CUtensorMap& map_w, const CUtensorMap& map_x, GemmArgs args, int forced_split,
                        cudaStream_t stream) {
   using Shape = GemmShape<kSwiglu, BN>;
-  auto kernel = gemm_bf16_kernel<kSwiglu, BN>;
-  bool& configured = g_gemm_configured[kSwiglu ? 1 : 0][BN / 32];
+  static_assert(!(kSwiglu && kRelu2), "one activation");
+  auto kernel = gemm_bf16_kernel<kSwiglu, BN, kRelu2>;
+  bool& configured = g_gemm_configured[kRelu2 ? 2 : (kSwiglu ? 1 : 0)][BN / 32];
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(Shape::kSmemBytes));
@@ -656,11 +662,14 @@ int rl_gemm_bf16_norm(const void* x, const void* w, void* out, int tokens, int n
   args.bias = bias;
   args.glu_limit = glu_limit; args.glu_alpha = glu_alpha;
   args.relu2_columns = relu2_columns; args.residual_scale = residual_scale;
-#define RL_GEMM_CASE(SW, BNV) \
-  if ((swiglu != 0) == SW && bn == BNV) return rl::launch_gemm<SW, BNV>(map_w, map_x, args, k_split, stream);
-  RL_GEMM_CASE(false, 16) RL_GEMM_CASE(false, 32) RL_GEMM_CASE(false, 64) RL_GEMM_CASE(false, 128)
-  RL_GEMM_CASE(false, 256) RL_GEMM_CASE(true, 16) RL_GEMM_CASE(true, 32) RL_GEMM_CASE(true, 64)
-  RL_GEMM_CASE(true, 128)
+#define RL_GEMM_CASE(SW, BNV, R2) \
+  if ((swiglu != 0) == SW && bn == BNV && (relu2_columns > 0) == R2) \
+    return rl::launch_gemm<SW, BNV, R2>(map_w, map_x, args, k_split, stream);
+  RL_GEMM_CASE(false, 16, false) RL_GEMM_CASE(false, 32, false) RL_GEMM_CASE(false, 64, false)
+  RL_GEMM_CASE(false, 128, false) RL_GEMM_CASE(false, 256, false) RL_GEMM_CASE(true, 16, false)
+  RL_GEMM_CASE(true, 32, false) RL_GEMM_CASE(true, 64, false) RL_GEMM_CASE(true, 128, false)
+  RL_GEMM_CASE(false, 16, true) RL_GEMM_CASE(false, 32, true) RL_GEMM_CASE(false, 64, true)
+  RL_GEMM_CASE(false, 128, true) RL_GEMM_CASE(false, 256, true)
 #undef RL_GEMM_CASE
   return static_cast<int>(cudaErrorInvalidValue);
 }
