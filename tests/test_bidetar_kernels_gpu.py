@@ -82,6 +82,24 @@ def test_the_square_of_relu_in_place_on_some_columns(width, stride, column, dtyp
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("width,before", [(48, 16), (13, 3)])
+def test_a_gate_entry_by_entry_into_the_columns_beside_it(width, before, dtype):
+    """The result goes to some columns of the rows that also hold the gate, as in a stack of products."""
+    from rapid_llm_b200.ops import kernels
+
+    g = torch.Generator().manual_seed(width)
+    rows = torch.randn(21, width, generator=g).to(dtype)
+    base = torch.randn(21, before + 2 * width + 8, generator=g).to(dtype)
+    wide = base.to(DEVICE)
+    gate = wide[:, before + width : before + 2 * width]
+    kernels.sigmoid_gate(rows.to(DEVICE), gate, wide[:, before : before + width])
+    want = rows.float() * torch.sigmoid(base[:, before + width : before + 2 * width].float())
+    bound = {"rtol": 1e-5, "atol": 1e-6} if dtype == torch.float32 else {"rtol": 1e-2, "atol": 1e-2}
+    torch.testing.assert_close(wide[:, before : before + width].float().cpu(), want, **bound)
+    assert torch.equal(wide[:, :before].cpu(), base[:, :before]) and torch.equal(wide[:, before + width :].cpu(), base[:, before + width :])
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("hidden", [64, 50, 1032])
 def test_what_joins_the_stream_is_weighed(hidden, dtype):
     """``residual <- residual + m * x`` in float32, and the norm of it; every row, and picked rows without storing."""
