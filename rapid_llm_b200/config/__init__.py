@@ -4,6 +4,7 @@ from .engine_config import EngineConfig, parse_dtype
 from .model_spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
 from .basitar import BasitarConfig
 from .bidetar import BidetarConfig
+from .danalorn import DanalornConfig
 from .kopatar import KopatarConfig
 from .mezadra import MezadraConfig
 from .qwen3 import Qwen3Config
@@ -22,10 +23,12 @@ register_architecture(MezadraConfig)
 register_architecture(BasitarConfig)
 register_architecture(ZupupelConfig)
 register_architecture(BidetarConfig)
+register_architecture(DanalornConfig)
 
 __all__ = [
     "BasitarConfig",
     "BidetarConfig",
+    "DanalornConfig",
     "EngineConfig",
     "KopatarConfig",
     "LayerSpec",

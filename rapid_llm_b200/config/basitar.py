@@ -27,7 +27,6 @@ from __future__ import annotations
 
 import copy
 from dataclasses import dataclass, field
-from pathlib import Path
 from typing import Any, Mapping
 
 from .model_spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
@@ -59,13 +58,9 @@ class BasitarConfig:
             if layer.get("type") != "wkv" or "decay_rank" in (layer.get("mixer") or {}):
                 continue
             if shapes is None:
-                from ..weights.safetensors_io import SafetensorsFile
+                from ..weights.safetensors_io import tensor_shapes
 
-                shapes = {}
-                for path in sorted(Path(model_dir).glob("*.safetensors")):
-                    handle = SafetensorsFile(path)
-                    shapes.update({name: handle.shape(name) for name in handle.keys()})
-                    handle.close()
+                shapes = tensor_shapes(model_dir)
             owner = layer.get("weights_of", index)
             name = f"l{owner}.mix.w1"
             if name not in shapes:

@@ -28,7 +28,7 @@
 //     through distributed shared memory, in rank order: no scratch in global memory and no
 //     second kernel.
 //
-// Semantics are those of attention_mma.cu, a sink and chunks included, squashed scores not (scores, running maximum and sum and the output
+// Semantics are those of attention_mma.cu, a sink, slopes and chunks included, squashed scores not (scores, running maximum and sum and the output
 // accumulator in float32; P rounded to bfloat16 before P.V).  Needs head size 128 and pages of
 // 8, 16, 32, 64 or a multiple of 128 tokens; everything else takes the mma.sync kernel.
 #pragma once
@@ -80,6 +80,7 @@ struct DecodeTcArgs {
   const bf16* gate;         // [tokens, hq] or null: a head's output is multiplied by sigmoid(gate)
   int gate_stride;
   const float* sink;        // [hq] float32 or null: exp(sink[head]) joins every row's denominator once
+  const float* slopes;      // [hq] float32 or null: slopes[head] * (query position - key position) is taken off every score
   int* fault;
 };
 
@@ -91,7 +92,7 @@ __device__ __forceinline__ float warp_max_redux(float v) {
 }
 
 // kRows: how many of the 16 columns of the products carry query rows (a power of two); the
-// per-row work of the softmax threads is unrolled over exactly these.  kDressed: the row's last step knows a sink, a
+// per-row work of the softmax threads is unrolled over exactly these.  kDressed: scores know slopes, the row's last step a sink, a
 // gate and an output whose rows are some columns of wider ones (the plain form keeps its registers and its short tail).
 template <int kRows, int kTcStages, bool kDressed>
 __global__ void __launch_bounds__(kTcThreads, kTcStages == 1 ? 2 : 1)
@@ -367,8 +368,13 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
 
     float prev_alpha[kRows];
     int pos_of[kRows], lo_of[kRows];
+    float slope_of[kDressed ? kRows : 1];                  // in base-2 units
 #pragma unroll
     for (int n = 0; n < kRows; ++n) {
+      if constexpr (kDressed) {
+        const int p = row0 + n;
+        slope_of[n] = args.slopes != nullptr && n < n_rows ? args.slopes[kv_head * group + p % group] * 1.4426950408889634f : 0.0f;
+      }
       pos_of[n] = row_pos[n];
       lo_of[n] = row_lo[n];
       prev_alpha[n] = 1.0f;
@@ -403,7 +409,9 @@ attention_decode_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const 
 #pragma unroll
       for (int n = 0; n < kRows; ++n) {
         const bool keep = in_range && key <= pos_of[n] && key >= lo_of[n];
-        s[n] = keep ? s[n] * args.scale_log2 : -INFINITY;
+        float scaled = s[n] * args.scale_log2;
+        if constexpr (kDressed) scaled = fmaf(slope_of[n], static_cast<float>(key - pos_of[n]), scaled);
+        s[n] = keep ? scaled : -INFINITY;
         const float m = warp_max_redux(s[n]);
         if (lane == 0) block_maxes[team][buf][quarter][n] = m;
       }

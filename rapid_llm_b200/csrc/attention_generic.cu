@@ -13,7 +13,8 @@
 // s_j = (q . k_j) * scale over the cached positions j <= p of the same request (and
 // j > p - window when a window is set: the query's own position counts, as in
 // rapid_llm/engine/kv_cache_spec.py:204,221-224; and j of the chunk p lies in when a chunk size is set); softmax over j; o = sum_j P_j v_j.
-// Scores, running maximum and sum, and the output accumulator are float32.
+// With slopes, slope[head] * (p - j) is taken off the score (after a cap).  Scores, running maximum and sum, and the
+// output accumulator are float32.
 #include "common.cuh"
 
 namespace rl {
@@ -33,7 +34,8 @@ __global__ void attention_generic_kernel(
     const int* __restrict__ token_slot, // [tokens]
     const int* __restrict__ block_table,  // [slots, max_pages]
     int tokens, int hq, int hkv, int d, int page_size, int num_pages, int max_pages, int slots,
-    int window, int chunk, float scale, float softcap, const float* __restrict__ sink, int kv_planes, int* __restrict__ fault) {
+    int window, int chunk, float scale, float softcap, const float* __restrict__ sink,
+    const float* __restrict__ slopes, int kv_planes, int* __restrict__ fault) {
   __shared__ float q_staged[kGenericWarps][kMaxD];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = static_cast<long long>(blockIdx.x) * kGenericWarps + warp;
@@ -56,6 +58,7 @@ __global__ void attention_generic_kernel(
   for (int i = lane; i < d; i += 32) qs[i] = to_float(qr[i]) * scale;
   __syncwarp();
 
+  const float slope = slopes != nullptr ? slopes[head] : 0.0f;
   const int first = first_visible(pos, window, chunk);
   const size_t head_stride = static_cast<size_t>(page_size) * d;
   // K plane -> V plane; a cache of one plane keeps rows that are keys and values at once
@@ -88,6 +91,7 @@ __global__ void attention_generic_kernel(
         }
         // squashed scores: cap * tanh(s / cap) of the scaled score, where the mixer has a cap
         score = softcap > 0.0f ? softcap * tanhf(dot / softcap) : dot;
+        score -= slope * static_cast<float>(pos - j);
       }
     }
     const float chunk_max = warp_max(score);
@@ -135,7 +139,7 @@ extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache,
                                     const int* positions, const int* token_slot,
                                     const int* block_table, int tokens, int hq, int hkv, int d,
                                     int page_size, int num_pages, int max_pages, int slots,
-                                    int window, int chunk, float scale, float softcap, const float* sink, int kv_planes,
+                                    int window, int chunk, float scale, float softcap, const float* sink, const float* slopes, int kv_planes,
                                     int* fault, cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (d <= 0 || d % 16 != 0 || d > rl::kGenericWideD || hkv <= 0 || hq % hkv != 0 ||
@@ -151,7 +155,7 @@ extern "C" int rl_attention_generic(int dtype, const void* q, const void* cache,
     kernel<<<blocks, rl::kGenericWarps * 32, 0, stream>>>(
         static_cast<const scalar_t*>(q), static_cast<const scalar_t*>(cache),
         static_cast<scalar_t*>(out), out_stride, static_cast<const scalar_t*>(gate), gate_stride, positions, token_slot, block_table, tokens, hq, hkv, d,
-        page_size, num_pages, max_pages, slots, window, chunk, scale, softcap, sink, kv_planes, fault);
+        page_size, num_pages, max_pages, slots, window, chunk, scale, softcap, sink, slopes, kv_planes, fault);
   });
   return rl::launch_status();
 }

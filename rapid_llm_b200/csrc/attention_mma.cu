@@ -19,7 +19,7 @@
 // rapid_llm/kernels/ops/attention/flashdecoding.py:223-230,335-407): kv head = q head //
 // group; s_j = (q . k_j) * scale for cached j <= p of the same request (and j > p - window
 // when a window is set; j of p's own chunk when a chunk size is set); softmax over j; o = sum_j P_j v_j.  Scores, running maximum and
-// sum and the output accumulator are float32; the exponent is taken in base 2 with log2(e)
+// sum and the output accumulator are float32 (with slopes, slope[head] * (p - j) is taken off the score); the exponent is taken in base 2 with log2(e)
 // folded into the scale; P is rounded to bfloat16 before the P.V product, as the
 // reference's tensor-core kernels do (flashattention2_nopad.py:162).
 #include <mutex>
@@ -72,6 +72,7 @@ struct AttentionArgs {
   float scale;              // the plain scale (used with softcap)
   float softcap;            // 0 = scores are not squashed
   const float* sink;        // null = no sink
+  const float* slopes;      // [hq] float32 or null: slopes[head] * (query position - key position) is taken off every score (caches of two planes)
   int out_stride;           // a multiple of 8
   const bf16* gate;         // [tokens, hq] (rows gate_stride apart) or null: a head's output is multiplied by its sigmoid
   int gate_stride;
@@ -117,7 +118,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // kWarpsM warps stacked over the tile's rows, kWarpsN warps side by side over each block's keys.
 // kShared: the cache has one plane, a row is key and value at once, and a block's rows are brought to shared
 // memory once and read as both (half the copies, half the stages' memory, so two CTAs fit on an SM at any head size).
-template <int kWarpsM, int kWarpsN, int kStages, bool kShared>
+// kSloped: a slope per head times the distance between query and key is taken off the score.
+template <int kWarpsM, int kWarpsN, int kStages, bool kShared, bool kSloped>
 __global__ void __launch_bounds__(kThreads)
 attention_mma_kernel(const AttentionArgs args) {
   static_assert(kWarpsM * kWarpsN == 4, "four warps");
@@ -155,6 +157,12 @@ attention_mma_kernel(const AttentionArgs args) {
     row_head[i] = kv_head * group + (p - token * group);
     row_pos[i] = row_valid[i] ? start + token : -1;
     row_lo[i] = first_visible(row_pos[i], args.window, args.chunk);
+  }
+  float slope_log2[2] = {0.0f, 0.0f};
+  if constexpr (kSloped) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (row_valid[i]) slope_log2[i] = args.slopes[row_head[i]] * 1.4426950408889634f;
   }
 
   const int last_row = min(n_rows, row0 + kTileM) - 1;
@@ -352,6 +360,7 @@ attention_mma_kernel(const AttentionArgs args) {
                     ? args.softcap * 1.4426950408889634f *
                           (1.0f - __fdividef(2.0f, 1.0f + exp2f(s[nt][e] * (2.8853900817779268f * args.scale / args.softcap))))
                     : s[nt][e] * args.scale_log2;
+            if constexpr (kSloped) v = fmaf(slope_log2[i], static_cast<float>(j - row_pos[i]), v);
           }
           s[nt][e] = v;
           block_max[i] = fmaxf(block_max[i], v);
@@ -537,9 +546,9 @@ constexpr size_t attention_smem_bytes() {
   return static_cast<size_t>(16 * kWarpsM + (kShared ? 1 : 2) * kStages * kBlockN) * kStride * sizeof(bf16);
 }
 
-template <int kWarpsM, int kWarpsN, int kStages, bool kShared>
+template <int kWarpsM, int kWarpsN, int kStages, bool kShared, bool kSloped>
 int launch_attention_as(const AttentionArgs& args, int n_items, bool pdl, cudaStream_t stream) {
-  auto kernel = attention_mma_kernel<kWarpsM, kWarpsN, kStages, kShared>;
+  auto kernel = attention_mma_kernel<kWarpsM, kWarpsN, kStages, kShared, kSloped>;
   constexpr size_t smem = attention_smem_bytes<kWarpsM, kWarpsN, kStages, kShared>();
   static_assert(smem <= 227 * 1024, "shared memory of one CTA");
   static bool configured = false;   // one per instantiation and per library image
@@ -554,8 +563,9 @@ int launch_attention_as(const AttentionArgs& args, int n_items, bool pdl, cudaSt
 
 template <int kWarpsM, int kWarpsN, int kStages>
 int launch_attention(const AttentionArgs& args, int n_items, bool pdl, cudaStream_t stream) {
-  return args.kv_planes == 1 ? launch_attention_as<kWarpsM, kWarpsN, kStages, true>(args, n_items, pdl, stream)
-                             : launch_attention_as<kWarpsM, kWarpsN, kStages, false>(args, n_items, pdl, stream);
+  if (args.kv_planes == 1) return launch_attention_as<kWarpsM, kWarpsN, kStages, true, false>(args, n_items, pdl, stream);
+  if (args.slopes != nullptr) return launch_attention_as<kWarpsM, kWarpsN, kStages, false, true>(args, n_items, pdl, stream);
+  return launch_attention_as<kWarpsM, kWarpsN, kStages, false, false>(args, n_items, pdl, stream);
 }
 
 }  // namespace RL_ATTENTION_NS
@@ -572,15 +582,16 @@ static bool decode_tc_supported(int page_size) {
   return kD == kTcD && page_size % 8 == 0 && (kTcKeys % page_size == 0 || page_size % kTcKeys == 0);
 }
 
-static bool g_prefill_tc_configured = false;   // file-local on purpose
+static bool g_prefill_tc_configured[2] = {};   // per instantiation; file-local on purpose
 
 // Chunk tiles of 256 packed rows on the tcgen05 kernel (unsplit key ranges only).
 static int launch_prefill_tc(const AttentionArgs& a, int n_items, bool pdl, cudaStream_t stream) {
-  if (!g_prefill_tc_configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         kPfSmemBytes);
+  const bool sloped = a.slopes != nullptr;
+  auto kernel = sloped ? attention_prefill_tc_kernel<true> : attention_prefill_tc_kernel<false>;
+  if (!g_prefill_tc_configured[sloped]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes);
     if (e != cudaSuccess) return static_cast<int>(e);
-    g_prefill_tc_configured = true;
+    g_prefill_tc_configured[sloped] = true;
   }
   CUtensorMap map;
   const long long rows = static_cast<long long>(a.num_pages) * 2 * a.hkv * a.page_size;
@@ -592,12 +603,12 @@ static int launch_prefill_tc(const AttentionArgs& a, int n_items, bool pdl, cuda
   t.page_size = a.page_size; t.num_pages = a.num_pages; t.max_pages = a.max_pages; t.slots = a.slots;
   t.window = a.window; t.chunk = a.chunk; t.scale_log2 = a.scale_log2; t.fault = a.fault;
   t.out_stride = a.out_stride; t.gate = a.gate; t.gate_stride = a.gate_stride;
-  t.softcap = a.softcap; t.sink = a.sink; t.cap_in = 0.0f; t.cap_out = 0.0f;
+  t.softcap = a.softcap; t.sink = a.sink; t.slopes = a.slopes; t.cap_in = 0.0f; t.cap_out = 0.0f;
   if (a.softcap > 0.0f) {
     t.cap_in = 2.0f * 1.4426950408889634f * a.scale / a.softcap;
     t.cap_out = a.softcap * 1.4426950408889634f;
   }
-  return launch_kernel(attention_prefill_tc_kernel, dim3(a.hkv, n_items), dim3(kPfThreads), kPfSmemBytes, stream, pdl,
+  return launch_kernel(kernel, dim3(a.hkv, n_items), dim3(kPfThreads), kPfSmemBytes, stream, pdl,
                        map, t);
 }
 
@@ -655,7 +666,7 @@ static int launch_decode_tc_as(const CUtensorMap& map, const DecodeTcArgs& t, in
 template <int kRows, int kStages>
 static int launch_decode_tc_stages(const CUtensorMap& map, const DecodeTcArgs& t, int n_items, bool pdl,
                                    cudaStream_t stream, bool* configured) {
-  const bool dressed = t.sink != nullptr || t.gate != nullptr || t.out_stride != t.hq * kTcD;
+  const bool dressed = t.sink != nullptr || t.slopes != nullptr || t.gate != nullptr || t.out_stride != t.hq * kTcD;
   if (dressed) return launch_decode_tc_as<kRows, kStages, true>(map, t, n_items, pdl, stream, configured + 1);
   return launch_decode_tc_as<kRows, kStages, false>(map, t, n_items, pdl, stream, configured);
 }
@@ -688,7 +699,7 @@ static int launch_decode_tc(const AttentionArgs& a, int n_items, int max_rows, b
   t.block_table = a.block_table; t.hq = a.hq; t.hkv = a.hkv; t.page_size = a.page_size;
   t.num_pages = a.num_pages; t.max_pages = a.max_pages; t.slots = a.slots; t.window = a.window;
   t.out_stride = a.out_stride; t.gate = a.gate; t.gate_stride = a.gate_stride;
-  t.chunk = a.chunk; t.sink = a.sink; t.splits = a.splits; t.cluster_merge = cluster_merge ? 1 : 0; t.scale_log2 = a.scale_log2; t.fault = a.fault;
+  t.chunk = a.chunk; t.sink = a.sink; t.slopes = a.slopes; t.splits = a.splits; t.cluster_merge = cluster_merge ? 1 : 0; t.scale_log2 = a.scale_log2; t.fault = a.fault;
   if (max_rows <= 0 || max_rows > kTcRows) max_rows = kTcRows;
   if (max_rows <= 1) return launch_decode_tc_rows<1>(map, t, n_items, pdl, stream, g_decode_tc_configured[0], rings);
   if (max_rows <= 2) return launch_decode_tc_rows<2>(map, t, n_items, pdl, stream, g_decode_tc_configured[1], rings);
@@ -754,7 +765,7 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
                      const int* entry_slot, const int* block_table, int tokens, int hq, int hkv,
                      int head_dim, int page_size, int num_pages, int max_pages, int slots,
                      int window, int chunk, int splits, float scale, int* fault, int pdl, int decode_kernel, int decode_rows,
-                     int chunk_rows, int decode_splits, float softcap, const float* sink, int kv_planes, int out_stride,
+                     int chunk_rows, int decode_splits, float softcap, const float* sink, const float* slopes, int kv_planes, int out_stride,
                      const void* gate, int gate_stride,
                      cudaStream_t stream) {
   if (tokens == 0 || (n_chunk_items == 0 && n_decode_items == 0)) return 0;
@@ -763,7 +774,7 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
     decode_kernel = 1;
   }
   if (kv_planes == 1) {         // rows that are keys and values at once: the mma.sync tiles read them, the tcgen05 tiles do not
-    if (chunk_rows == attn::kPfRows || (decode_splits > 0 && decode_splits != splits)) return static_cast<int>(cudaErrorInvalidValue);
+    if (slopes != nullptr || chunk_rows == attn::kPfRows || (decode_splits > 0 && decode_splits != splits)) return static_cast<int>(cudaErrorInvalidValue);
     decode_kernel = 1;
   } else if (kv_planes != 2) {
     return static_cast<int>(cudaErrorInvalidValue);
@@ -795,7 +806,7 @@ int rl_attention_mma(const void* q, const void* cache, void* out, float* part_ou
   args.max_pages = max_pages; args.slots = slots; args.window = window; args.chunk = chunk; args.splits = splits;
   args.scale_log2 = scale * 1.4426950408889634f;
   args.fault = fault;
-  args.scale = scale; args.softcap = softcap; args.sink = sink; args.kv_planes = kv_planes;
+  args.scale = scale; args.softcap = softcap; args.sink = sink; args.slopes = slopes; args.kv_planes = kv_planes;
   args.out_stride = out_stride; args.gate = static_cast<const attn::bf16*>(gate); args.gate_stride = gate_stride;
   int status = 0;
   bool merged_in_cluster = false;
@@ -923,7 +934,7 @@ int rl_attention_mma_static_scratch(const void* q, const void* cache, void* out,
   }
   return rl_attention_mma(q, cache, out, part_out, part_lse, chunk_items, n_chunk_items, decode_items,
                           n_decode_items, cu_seqlens, entry_start, entry_slot, block_table, tokens, hq, hkv,
-                          head_dim, page_size, num_pages, max_pages, slots, window, 0, splits, scale, fault, 0, 1, 0, 64, 0, 0.0f, nullptr, 2,
+                          head_dim, page_size, num_pages, max_pages, slots, window, 0, splits, scale, fault, 0, 1, 0, 64, 0, 0.0f, nullptr, nullptr, 2,
                           hq * head_dim, nullptr, 0, stream);
 }
 

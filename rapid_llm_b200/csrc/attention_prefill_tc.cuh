@@ -96,6 +96,7 @@ struct PrefillTcArgs {
   // cap_out * (1 - 2 / (1 + 2^(raw * cap_in))), cap_in = 2 log2(e) scale / softcap, cap_out = softcap log2(e).
   float softcap, cap_in, cap_out;
   const float* sink;
+  const float* slopes;      // [hq] float32 or null: slopes[head] * (query position - key position) is taken off every score
   int out_stride;           // elements from a token's row of out to the next
   const bf16* gate;         // [tokens, hq] or null: a head's output is multiplied by sigmoid(gate)
   int gate_stride;
@@ -107,6 +108,8 @@ __device__ __forceinline__ float pf_fast_rcp(float x) {
   return y;
 }
 
+// kSloped: `slopes` is given (the plain form keeps its registers and its one multiply-add per score).
+template <bool kSloped>
 __global__ void __launch_bounds__(kPfThreads, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const PrefillTcArgs args) {
   extern __shared__ unsigned char pf_smem_raw[];
@@ -367,7 +370,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const
 
     const int my_blocks = tile_blocks[tile];
     const bool capped = args.softcap > 0.0f;           // the same for every thread of the grid
-    const float post_scale = capped ? 1.0f : args.scale_log2;
+    const float post_scale = capped || kSloped ? 1.0f : args.scale_log2;
+    float slope_log2 = 0.0f;
+    if constexpr (kSloped) {
+      if (valid) slope_log2 = args.slopes[kv_head * group + (p - token * group)] * 1.4426950408889634f;
+    }
     float ref_max = -INFINITY;                         // exponentials are taken against ref_max
     unsigned long long row_sum2 = pf_pack2(0.0f, 0.0f);   // the row's sum as two halves (even and odd keys)
     bool ok = true;
@@ -391,6 +398,23 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_cache, const
           const float raw = __uint_as_float(score[i >> 5][i & 31]);
           const float squashed = fmaf(-2.0f * args.cap_out, pf_fast_rcp(1.0f + fast_exp2(raw * args.cap_in)), args.cap_out);
           score[i >> 5][i & 31] = __float_as_uint(squashed);
+        }
+      }
+      if constexpr (kSloped) {
+        // base-2 score plus slope * (key - pos), two keys an instruction: the block's first distance joins with the scale,
+        // the places inside the block are constants
+        const float in_scale = capped ? 1.0f : args.scale_log2;
+        const float nearest = slope_log2 * static_cast<float>(kb - pos);
+        const unsigned long long in2 = pf_pack2(in_scale, in_scale), slope2 = pf_pack2(slope_log2, slope_log2);
+        const unsigned long long nearest2 = pf_pack2(nearest, nearest);
+#pragma unroll
+        for (int i = 0; i < kPfKeys; i += 2) {
+          const unsigned long long at2 = pf_pack2(static_cast<float>(i), static_cast<float>(i + 1));
+          const unsigned long long bias2 = pf_fma2(slope2, at2, nearest2);
+          float x0, x1;
+          pf_unpack2(pf_fma2(pf_pack2(__uint_as_float(score[i >> 5][i & 31]), __uint_as_float(score[(i + 1) >> 5][(i + 1) & 31])), in2, bias2), x0, x1);
+          score[i >> 5][i & 31] = __float_as_uint(x0);
+          score[(i + 1) >> 5][(i + 1) & 31] = __float_as_uint(x1);
         }
       }
       if (masked) {

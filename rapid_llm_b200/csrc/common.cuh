@@ -110,6 +110,11 @@ __device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
   return window > 0 ? max(0, pos - window + 1) : 0;
 }
 
+// A query's temperature at `pos`: 1 + coef * ln(floor((pos + 1) / every) + 1).
+__device__ __forceinline__ float query_temperature(int pos, float coef, float every) {
+  return 1.0f + coef * logf(floorf(__fdiv_rn(static_cast<float>(pos + 1), every)) + 1.0f);
+}
+
 // A gate of one number per token and head, applied to a head's output: sigmoid(gate[token * stride + head]), or 1
 // without a gate.
 template <typename T>

@@ -78,7 +78,7 @@ __global__ void embedding_sum_kernel(T* __restrict__ out, float* __restrict__ st
                                      const int* __restrict__ positions, const int* __restrict__ cu_seqlens,
                                      const int* __restrict__ entry_slot, int entries, int* last_token, int slots,
                                      int hidden, int vocab, int buckets, long long mul_prev, long long mul_cur,
-                                     int max_positions, int* __restrict__ fault) {
+                                     int max_positions, float scale, int* __restrict__ fault) {
   pdl_trigger();
   const int t = blockIdx.x;
   auto id_of = [&](int row) {
@@ -95,7 +95,7 @@ __global__ void embedding_sum_kernel(T* __restrict__ out, float* __restrict__ st
   int slot = entry_slot[e];
   const bool slot_ok = slot >= 0 && slot < slots;
   int pos = positions[t];
-  if (pos < 0 || pos >= max_positions) {
+  if (pos < 0 || (position_table != nullptr && pos >= max_positions)) {
     if (threadIdx.x == 0) atomicOr(fault, kFaultPosition);
     pos = 0;
   }
@@ -111,12 +111,13 @@ __global__ void embedding_sum_kernel(T* __restrict__ out, float* __restrict__ st
   if (t == first && slot_ok && threadIdx.x == 0) last_token[slot] = id_of(last);
   const T* a = table + static_cast<size_t>(id) * hidden;
   const T* b = pair_table + static_cast<size_t>(row) * hidden;
-  const T* c = position_table + static_cast<size_t>(pos) * hidden;
+  const T* c = position_table == nullptr ? nullptr : position_table + static_cast<size_t>(pos) * hidden;
   T* dst = out + static_cast<size_t>(t) * hidden;
   float* sr = stream ? stream + static_cast<size_t>(t) * hidden : nullptr;
   pdl_wait();
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-    const float v = to_float(a[i]) + to_float(b[i]) + to_float(c[i]);
+    float v = scale * to_float(a[i]) + to_float(b[i]);
+    if (c != nullptr) v += to_float(c[i]);
     if (sr) sr[i] = v;
     dst[i] = from_float<T>(v);
   }
@@ -508,7 +509,7 @@ int rl_embedding_sum(int dtype, void* out, float* stream_out, const void* table,
                      const void* position_table, const int* ids, const int* feedback, int feedback_rows,
                      const int* positions, const int* cu_seqlens, const int* entry_slot, int entries, int* last_token,
                      int slots, int rows, int hidden, int vocab, int buckets, long long mul_prev, long long mul_cur,
-                     int max_positions, int* fault, cudaStream_t stream) {
+                     int max_positions, float scale, int* fault, cudaStream_t stream) {
   if (rows == 0) return 0;
   if (entries < 1 || buckets < 1 || hidden < 1) return static_cast<int>(cudaErrorInvalidValue);
   RL_DISPATCH_DTYPE(dtype, {
@@ -517,7 +518,7 @@ int rl_embedding_sum(int dtype, void* out, float* stream_out, const void* table,
                              static_cast<scalar_t*>(out), stream_out, static_cast<const scalar_t*>(table),
                              static_cast<const scalar_t*>(pair_table), static_cast<const scalar_t*>(position_table),
                              ids, feedback, feedback_rows, positions, cu_seqlens, entry_slot, entries, last_token, slots,
-                             hidden, vocab, buckets, mul_prev, mul_cur, max_positions, fault);
+                             hidden, vocab, buckets, mul_prev, mul_cur, max_positions, scale, fault);
   });
   return 0;
 }

@@ -22,14 +22,14 @@ __device__ __forceinline__ void pair_places(int i, int rot, int layout, int& lo,
 
 // ------------------------------------------------------------ norms of the two latents, the cache row
 // One block per token.  `down` holds [query latent (q_rank) | ... | c (kv_rank) | key part (rot)] at the given
-// columns (q_rank 0: there is no query latent, and q_out is not touched).  q_out = RMS norm of the query latent with
+// columns (q_rank 0: there is no query latent, and q_out is not touched; cache null: the layer reads another one's
+// rows, and there is no c).  q_out = RMS norm of the query latent with
 // weight wq; the cache row at kv_dest[t] receives
 // [RMS norm of c with weight wc | rotated key part | zeros up to D].
 template <typename T>
-__global__ void latent_norm_write_kernel(const T* __restrict__ down, int down_stride, int q_col0, int q_rank,
+__global__ void latent_norm_write_kernel(const T* down, int down_stride, int q_col0, int q_rank,
                                          int c_col0, int kv_rank, int rot, const float* __restrict__ wq,
-                                         const float* __restrict__ wc, float eps, T* __restrict__ q_out,
-                                         T* __restrict__ cache, const int* __restrict__ kv_dest, long long cache_rows,
+                                         const float* __restrict__ wc, float eps, T* q_out, T* cache, const int* __restrict__ kv_dest, long long cache_rows,
                                          int D, const int* __restrict__ positions, const float* __restrict__ freq,
                                          float magnitude, int layout, int* __restrict__ fault) {
   __shared__ float scratch[32];
@@ -42,9 +42,11 @@ __global__ void latent_norm_write_kernel(const T* __restrict__ down, int down_st
     const float v = to_float(row[q_col0 + i]);
     sum_q += v * v;
   }
-  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) {
-    const float v = to_float(row[c_col0 + i]);
-    sum_c += v * v;
+  if (cache != nullptr) {
+    for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) {
+      const float v = to_float(row[c_col0 + i]);
+      sum_c += v * v;
+    }
   }
   sum_q = block_sum(sum_q, scratch);
   sum_c = block_sum(sum_c, scratch);
@@ -52,6 +54,7 @@ __global__ void latent_norm_write_kernel(const T* __restrict__ down, int down_st
   const float inv_c = rsqrtf(sum_c / static_cast<float>(kv_rank) + eps);
   T* qo = q_out + static_cast<size_t>(t) * q_rank;
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x) qo[i] = from_float<T>(to_float(row[q_col0 + i]) * inv_q * wq[i]);
+  if (cache == nullptr) return;
   const long long dest = kv_dest[t];
   if (dest < 0 || dest >= cache_rows) {
     if (threadIdx.x == 0) atomicOr(fault, kFaultPageId);
@@ -77,8 +80,7 @@ __global__ void latent_norm_write_kernel(const T* __restrict__ down, int down_st
 // q: [T, heads * (dim + rot)], a head's last `rot` numbers are its rotated part.  wide: [T, heads * D]; a head's
 // columns [kv_rank, kv_rank + rot) receive the rotation, the columns behind them zeros.  One block per token.
 template <typename T>
-__global__ void latent_rotate_queries_kernel(const T* __restrict__ q, int heads, int dim, int rot,
-                                             T* __restrict__ wide, int kv_rank, int D,
+__global__ void latent_rotate_queries_kernel(const T* q, int heads, int dim, int rot, T* wide, int kv_rank, int D,
                                              const int* __restrict__ positions, const float* __restrict__ freq,
                                              float magnitude, int layout) {
   pdl_trigger();
@@ -252,7 +254,7 @@ int rl_latent_norm_write(int dtype, const void* down, int down_stride, int q_col
                          float magnitude, int layout, int tokens, int* fault, int pdl, cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (q_rank < 0 || kv_rank < 1 || rot < 0 || rot % 2 || kv_rank + rot > D || layout < 0 || layout > 1 ||
-      (rot > 0 && freq == nullptr))
+      (rot > 0 && freq == nullptr) || (cache != nullptr && (kv_dest == nullptr || wc == nullptr)))
     return static_cast<int>(cudaErrorInvalidValue);
   RL_DISPATCH_DTYPE(dtype, {
     return rl::launch_kernel(rl::latent_norm_write_kernel<scalar_t>, dim3(tokens), dim3(128), 0, stream, pdl != 0,

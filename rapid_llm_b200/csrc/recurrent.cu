@@ -260,6 +260,102 @@ __global__ void exp_decay_kernel(const T* x, int x_stride, int col0, const float
   }
 }
 
+// ------------------------------------------------------------ decay from a low-rank product
+// decay[t, c] = sigmoid(bias[c] + sum_r w[c, r] low[t, r]) ^ (1 / tau), taken as exp(-softplus(-z) / tau): the second
+// product of a low-rank pair, its bias and the decay in one pass, in float32 from the stored numbers on (z is never
+// rounded).  Beside it the mixer's q, k and v columns as float32 rows, which the recurrence reads.  low and the copied
+// columns are columns of the same rows x.
+// A block takes kDecayTokens rows and kDecayThreads decays or 4 * kDecayThreads copied columns (the later blocks of the
+// y dimension); a decay's weight row is read once for its tokens.
+constexpr int kDecayThreads = 128;
+constexpr int kDecayTokens = 8;
+constexpr int kDecayRankStep = 32;      // numbers of a weight row held in registers at a time
+
+template <typename T>
+__global__ void __launch_bounds__(kDecayThreads) low_rank_decay_kernel(
+    const T* x, int x_stride, int copied, int low_col0, const T* __restrict__ w, int rank, const float* __restrict__ bias,
+    float inv_tau, float* rows, int channels, float* decay, int tokens, int decay_blocks, int vector_rows) {
+  __shared__ float low[kDecayTokens][kDecayRankStep];
+  pdl_trigger();
+  const int t0 = blockIdx.x * kDecayTokens, count = min(kDecayTokens, tokens - t0);
+  if (static_cast<int>(blockIdx.y) >= decay_blocks) {
+    const int c0 = ((blockIdx.y - decay_blocks) * kDecayThreads + threadIdx.x) * 4;
+    pdl_wait();
+    if (c0 >= copied) return;
+    if (vector_rows) {
+      // (eight loads in flight, then eight stores)
+      float4 v[kDecayTokens];
+#pragma unroll
+      for (int i = 0; i < kDecayTokens; ++i) {
+        if (i >= count) break;
+        const T* from = x + static_cast<size_t>(t0 + i) * x_stride + c0;
+        if constexpr (sizeof(T) == 2) {
+          const uint2 packed = *reinterpret_cast<const uint2*>(from);
+          const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&packed);
+          const float2 lo = __bfloat1622float2(h[0]), hi = __bfloat1622float2(h[1]);
+          v[i] = make_float4(lo.x, lo.y, hi.x, hi.y);
+        } else {
+          v[i] = *reinterpret_cast<const float4*>(from);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < kDecayTokens; ++i) {
+        if (i >= count) break;
+        *reinterpret_cast<float4*>(rows + static_cast<size_t>(t0 + i) * copied + c0) = v[i];
+      }
+      return;
+    }
+    for (int i = 0; i < count; ++i)
+      for (int c = c0; c < min(c0 + 4, copied); ++c)
+        rows[static_cast<size_t>(t0 + i) * copied + c] = to_float(x[static_cast<size_t>(t0 + i) * x_stride + c]);
+    return;
+  }
+  const int c = blockIdx.y * kDecayThreads + threadIdx.x;
+  const bool mine = c < channels;
+  float sum[kDecayTokens];
+#pragma unroll
+  for (int i = 0; i < kDecayTokens; ++i) sum[i] = mine ? bias[c] : 0.0f;
+  bool waited = false;
+  for (int r0 = 0; r0 < rank; r0 += kDecayRankStep) {
+    const int here = min(kDecayRankStep, rank - r0);
+    float wr[kDecayRankStep];
+    const T* from = w + static_cast<size_t>(mine ? c : 0) * rank + r0;
+    if (here == kDecayRankStep && rank % 8 == 0) {      // rows of whole 16-byte pieces (weights are aligned)
+#pragma unroll
+      for (int r = 0; r < kDecayRankStep; r += 8) {
+        float eight[8];
+        load8(from + r, eight);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) wr[r + j] = eight[j];
+      }
+    } else {
+#pragma unroll
+      for (int r = 0; r < kDecayRankStep; ++r) wr[r] = r < here ? to_float(from[r]) : 0.0f;
+    }
+    if (!waited) {
+      pdl_wait();
+      waited = true;
+    }
+    __syncthreads();
+    for (int idx = threadIdx.x; idx < kDecayTokens * kDecayRankStep; idx += kDecayThreads) {
+      const int i = idx / kDecayRankStep, r = idx - i * kDecayRankStep;
+      low[i][r] = i < count && r < here ? to_float(x[static_cast<size_t>(t0 + i) * x_stride + low_col0 + r0 + r]) : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kDecayTokens; ++i) {
+      if (i < count) {
+#pragma unroll
+        for (int r = 0; r < kDecayRankStep; ++r) sum[i] = fmaf(wr[r], low[i][r], sum[i]);
+      }
+    }
+  }
+  if (!mine) return;
+#pragma unroll
+  for (int i = 0; i < kDecayTokens; ++i)
+    if (i < count) decay[static_cast<size_t>(t0 + i) * channels + c] = expf(-softplus_f(-sum[i]) * inv_tau);
+}
+
 // ------------------------------------------------------------ tanh of rows, in the rows' own type
 // out[i] = tanh(x[i]) in float32, rounded once: the activation between the two halves of a low-rank product.
 template <typename T>
@@ -981,6 +1077,26 @@ int rl_exp_decay(int dtype, const void* x, int x_stride, int col0, const float* 
     return rl::launch_kernel(rl::exp_decay_kernel<scalar_t>,
                              dim3(rl::flat_blocks(static_cast<long long>(tokens) * channels, 256)), dim3(256), 0, stream,
                              pdl != 0, static_cast<const scalar_t*>(x), x_stride, col0, bias, decay, tokens, channels);
+  });
+  return 0;
+}
+
+int rl_low_rank_decay(int dtype, const void* x, int x_stride, int copied, int low_col0, const void* w, int rank,
+                      const float* bias, float tau, float* rows, int channels, float* decay, int tokens, int pdl,
+                      cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  if (rank < 1 || channels < 1 || copied < 0 || copied > x_stride || low_col0 < 0 || low_col0 + rank > x_stride || !(tau > 0.0f) ||
+      bias == nullptr || w == nullptr || (reinterpret_cast<uintptr_t>(w) & 15))
+    return static_cast<int>(cudaErrorInvalidValue);
+  const int decay_blocks = (channels + rl::kDecayThreads - 1) / rl::kDecayThreads;
+  const int copy_blocks = (copied + 4 * rl::kDecayThreads - 1) / (4 * rl::kDecayThreads);
+  const int vector_rows = copied % 4 == 0 && x_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 &&
+                          (reinterpret_cast<uintptr_t>(rows) & 15) == 0;
+  const dim3 grid((tokens + rl::kDecayTokens - 1) / rl::kDecayTokens, decay_blocks + copy_blocks);
+  RL_DISPATCH_DTYPE(dtype, {
+    return rl::launch_kernel(rl::low_rank_decay_kernel<scalar_t>, grid, dim3(rl::kDecayThreads), 0, stream, pdl != 0,
+                             static_cast<const scalar_t*>(x), x_stride, copied, low_col0, static_cast<const scalar_t*>(w), rank, bias,
+                             1.0f / tau, rows, channels, decay, tokens, decay_blocks, vector_rows);
   });
   return 0;
 }

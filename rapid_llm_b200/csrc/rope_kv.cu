@@ -30,17 +30,20 @@ struct RopeArgs {
   int tokens, row_width, hq, hkv, d, rotary, max_pos, page_size, num_pages;
   int norm_size;            // entries the norm's mean is taken over (d, or fewer when the head's tail is padding)
   float eps;
+  float temp_coef, temp_every;   // temp_every > 0: queries are multiplied by query_temperature(position, coef, every)
   int* fault;
 };
 
 // One warp per (token, run of heads).  kVec > 0: the head size is 32 * kVec, the whole head
-// rotates (rotary == d), and lane l holds the kVec consecutive elements from l * kVec in
+// rotates (rotary == d; kDressed: or nothing does), and lane l holds the kVec consecutive elements from l * kVec in
 // registers; its rotation partner (element + d/2) sits in lane l ^ 16.  A warp then takes
 // `heads_per_warp` consecutive heads of its token and fetches the token's angles and the norm
 // weights once for all of them (many heads a warp when there are many tokens, one when there
 // are few and the work has to spread over the SMs).  kVec == 0: any head size up to 256 and
 // any even rotary width, one head a warp, element by element through shared memory.
-template <typename T, int kVec>
+// kDressed: heads may pass without a rotation, and queries may have a temperature that depends on the position
+// (kVec == 0 knows both at run time).
+template <typename T, int kVec, bool kDressed>
 __global__ void qk_norm_rope_write_kernel(const RopeArgs a, const int heads_per_warp) {
   __shared__ float staged[kVec == 0 ? kRopeWarps : 1][kVec == 0 ? kMaxHeadDim : 1];
   pdl_trigger();
@@ -75,11 +78,13 @@ __global__ void qk_norm_rope_write_kernel(const RopeArgs a, const int heads_per_
   if constexpr (kVec > 0) {
     const int at = lane * kVec;
     const int angle = at < half ? at : at - half;      // kVec divides d / 2, so a lane never straddles
+    const bool rotates = !kDressed || half > 0;
+    const float warmth = kDressed && a.temp_every > 0.0f ? query_temperature(pos, a.temp_coef, a.temp_every) : 1.0f;
     float c[kVec], s[kVec], qw[kVec], kw[kVec];
 #pragma unroll
     for (int i = 0; i < kVec; ++i) {
-      c[i] = a.cos_table[static_cast<size_t>(pos) * half + angle + i];
-      s[i] = a.sin_table[static_cast<size_t>(pos) * half + angle + i];
+      c[i] = rotates ? a.cos_table[static_cast<size_t>(pos) * half + angle + i] : 1.0f;
+      s[i] = rotates ? a.sin_table[static_cast<size_t>(pos) * half + angle + i] : 0.0f;
       qw[i] = a.q_weight ? a.q_weight[at + i] : 1.0f;
       kw[i] = a.k_weight ? a.k_weight[at + i] : 1.0f;
     }
@@ -129,11 +134,19 @@ __global__ void qk_norm_rope_write_kernel(const RopeArgs a, const int heads_per_
 #pragma unroll
           for (int i = 0; i < kVec; ++i) v[i] = v[i] * inv_rms * (kind == 0 ? qw[i] : kw[i]);
         }
+        if (rotates) {
 #pragma unroll
-        for (int i = 0; i < kVec; ++i) {
-          const float other = __shfl_xor_sync(0xffffffffu, v[i], 16);
-          // first half: x1 * c - x2 * s; second half: x2 * c + x1 * s
-          v[i] = lane < 16 ? v[i] * c[i] - other * s[i] : v[i] * c[i] + other * s[i];
+          for (int i = 0; i < kVec; ++i) {
+            const float other = __shfl_xor_sync(0xffffffffu, v[i], 16);
+            // first half: x1 * c - x2 * s; second half: x2 * c + x1 * s
+            v[i] = lane < 16 ? v[i] * c[i] - other * s[i] : v[i] * c[i] + other * s[i];
+          }
+        }
+        if constexpr (kDressed) {
+          if (kind == 0) {
+#pragma unroll
+            for (int i = 0; i < kVec; ++i) v[i] *= warmth;
+          }
         }
       }
       if constexpr (kVec == 8) {
@@ -209,6 +222,7 @@ __global__ void qk_norm_rope_write_kernel(const RopeArgs a, const int heads_per_
     __syncwarp();
     const float* c = a.cos_table + static_cast<size_t>(pos) * half;
     const float* s = a.sin_table + static_cast<size_t>(pos) * half;
+    const float warmth = kind == 0 && a.temp_every > 0.0f ? query_temperature(pos, a.temp_coef, a.temp_every) : 1.0f;
     for (int i = lane; i < d; i += 32) {
       float v;
       if (i < half) {
@@ -218,7 +232,7 @@ __global__ void qk_norm_rope_write_kernel(const RopeArgs a, const int heads_per_
       } else {
         v = mine[i];
       }
-      dst[i] = from_float<T>(v);
+      dst[i] = from_float<T>(v * warmth);
     }
   }
 }
@@ -229,7 +243,9 @@ __global__ void qk_norm_rope_write_kernel(const RopeArgs a, const int heads_per_
 // the rotation needs no exchange between lanes and four angles a lane.  The kernel is bound by the bytes
 // it keeps in flight and by instruction issue, not by arithmetic: it stays within 64 registers (eight CTAs,
 // 32 warps a multiprocessor), asks for its heads before its angles (both wait on the position alone) and
-// reads the norm weights where it uses them (they stay in L1).
+// reads the norm weights where it uses them (they stay in L1).  kDressed: heads may pass without a rotation, and queries
+// may have a temperature.
+template <bool kDressed>
 __global__ void __launch_bounds__(kRopeWarps * 32, 8) qk_norm_rope_write_pairs_kernel(const RopeArgs a) {
   using T = __nv_bfloat16;
   constexpr int kHeadsPerWarp = 8, kD = 128, kHalf = kD / 2;
@@ -265,7 +281,9 @@ __global__ void __launch_bounds__(kRopeWarps * 32, 8) qk_norm_rope_write_pairs_k
     pos = 0;
   }
   float4 c = make_float4(1.0f, 1.0f, 1.0f, 1.0f), s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-  if (head_begin < a.hq + a.hkv) {                             // a warp of values alone needs no angles
+  const bool rotates = !kDressed || a.rotary > 0;
+  const float warmth = kDressed && a.temp_every > 0.0f ? query_temperature(pos, a.temp_coef, a.temp_every) : 1.0f;
+  if (rotates && head_begin < a.hq + a.hkv) {                  // a warp of values alone needs no angles
     c = __ldg(reinterpret_cast<const float4*>(a.cos_table + static_cast<size_t>(pos) * kHalf + at));
     s = __ldg(reinterpret_cast<const float4*>(a.sin_table + static_cast<size_t>(pos) * kHalf + at));
   }
@@ -329,6 +347,12 @@ __global__ void __launch_bounds__(kRopeWarps * 32, 8) qk_norm_rope_write_pairs_k
       for (int i = 0; i < 4; ++i) {
         o1[i] = x1[i] * cs[i] - x2[i] * sn[i];
         o2[i] = x2[i] * cs[i] + x1[i] * sn[i];
+        if constexpr (kDressed) {
+          if (kind == 0) {
+            o1[i] *= warmth;
+            o2[i] *= warmth;
+          }
+        }
       }
       __nv_bfloat162* h1 = reinterpret_cast<__nv_bfloat162*>(&out1);
       __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&out2);
@@ -351,10 +375,12 @@ extern "C" int rl_qk_norm_rope_write(int dtype, const void* qkv, int row_width, 
                                      const int* positions, const int* kv_dest, void* q_out,
                                      void* cache, int tokens, int hq, int hkv, int d, int rotary,
                                      int max_pos, int page_size, int num_pages, float eps,
-                                     int norm_size, int* fault, int pdl, cudaStream_t stream) {
+                                     int norm_size, float temp_coef, float temp_every, int* fault, int pdl,
+                                     cudaStream_t stream) {
   if (tokens == 0) return 0;
   if (d > rl::kMaxHeadDim || d <= 0 || rotary < 0 || rotary > d || (rotary & 1) ||
-      (kv_dest != nullptr && cache == nullptr) || norm_size < 0 || norm_size > d)
+      (kv_dest != nullptr && cache == nullptr) || norm_size < 0 || norm_size > d || temp_every < 0.0f ||
+      row_width < (kv_dest ? hq + 2 * hkv : hq) * d)
     return static_cast<int>(cudaErrorInvalidValue);
   const int heads_per_token = kv_dest ? hq + 2 * hkv : hq;
   rl::RopeArgs a;
@@ -363,10 +389,13 @@ extern "C" int rl_qk_norm_rope_write(int dtype, const void* qkv, int row_width, 
   a.q_out = q_out; a.cache = cache; a.tokens = tokens; a.row_width = row_width; a.hq = hq; a.hkv = hkv;
   a.d = d; a.rotary = rotary; a.max_pos = max_pos; a.page_size = page_size; a.num_pages = num_pages;
   a.eps = eps; a.fault = fault; a.norm_size = norm_size > 0 ? norm_size : d;
-  // registers when the whole head rotates, a lane's elements are whole vectors and everything is aligned
+  a.temp_coef = temp_coef; a.temp_every = temp_every;
+  // registers when the whole head rotates (or nothing of it), a lane's elements are whole vectors and everything is aligned
   const bool aligned = ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(q_out) |
                          reinterpret_cast<uintptr_t>(cache)) & 15) == 0 && row_width % 8 == 0;
-  const int vec = (rotary == d && d % 32 == 0 && aligned) ? d / 32 : 0;
+  const bool dressed = rotary == 0 || temp_every > 0.0f;
+  int vec = ((rotary == d || rotary == 0) && d % 32 == 0 && aligned) ? d / 32 : 0;
+  if (vec != 1 && vec != 2 && vec != 4 && vec != 8) vec = 0;      // (96 and its like have no register form)
   // a warp takes several heads of a token once there are enough tokens to fill the GPU anyway
   // (the kernel for heads of 128 in bfloat16, which keeps more bytes in flight, from about 200 tokens of 48 heads
   // on: measured equal below, 15 us faster at 512 tokens and 26 us at 1,024)
@@ -379,13 +408,13 @@ extern "C" int rl_qk_norm_rope_write(int dtype, const void* qkv, int row_width, 
   const bool tables_aligned = ((reinterpret_cast<uintptr_t>(cos_table) | reinterpret_cast<uintptr_t>(sin_table) |
                                 reinterpret_cast<uintptr_t>(q_weight) | reinterpret_cast<uintptr_t>(k_weight)) & 15) == 0;
   if (heads_per_warp == 8 && pairs_kernel && tables_aligned)
-    return rl::launch_kernel(rl::qk_norm_rope_write_pairs_kernel, grid, block, 0, stream, pdl != 0, a);
+    return rl::launch_kernel(dressed ? rl::qk_norm_rope_write_pairs_kernel<true> : rl::qk_norm_rope_write_pairs_kernel<false>, grid, block, 0, stream, pdl != 0, a);
   RL_DISPATCH_DTYPE(dtype, {
-    if (vec == 8) return rl::launch_kernel(rl::qk_norm_rope_write_kernel<scalar_t, 8>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
-    if (vec == 4) return rl::launch_kernel(rl::qk_norm_rope_write_kernel<scalar_t, 4>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
-    if (vec == 2) return rl::launch_kernel(rl::qk_norm_rope_write_kernel<scalar_t, 2>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
-    if (vec == 1) return rl::launch_kernel(rl::qk_norm_rope_write_kernel<scalar_t, 1>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
-    return rl::launch_kernel(rl::qk_norm_rope_write_kernel<scalar_t, 0>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
+    if (vec == 8) return rl::launch_kernel(dressed ? rl::qk_norm_rope_write_kernel<scalar_t, 8, true> : rl::qk_norm_rope_write_kernel<scalar_t, 8, false>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
+    if (vec == 4) return rl::launch_kernel(dressed ? rl::qk_norm_rope_write_kernel<scalar_t, 4, true> : rl::qk_norm_rope_write_kernel<scalar_t, 4, false>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
+    if (vec == 2) return rl::launch_kernel(dressed ? rl::qk_norm_rope_write_kernel<scalar_t, 2, true> : rl::qk_norm_rope_write_kernel<scalar_t, 2, false>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
+    if (vec == 1) return rl::launch_kernel(dressed ? rl::qk_norm_rope_write_kernel<scalar_t, 1, true> : rl::qk_norm_rope_write_kernel<scalar_t, 1, false>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
+    return rl::launch_kernel(rl::qk_norm_rope_write_kernel<scalar_t, 0, true>, grid, block, 0, stream, pdl != 0, a, heads_per_warp);
   });
   return 0;
 }

@@ -137,15 +137,16 @@ def core() -> ctypes.CDLL:
         lib.rl_qk_norm_rope_write.argtypes = [
             c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-            c_float, c_int, c_void_p, c_int, c_void_p,
+            c_float, c_int, c_float, c_float, c_void_p, c_int, c_void_p,
         ]
         lib.rl_attention_generic.argtypes = [
             c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p,
+            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
         ]
         lib.rl_embedding_sum.argtypes = [
             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_void_p, c_void_p,
+            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_float,
+            c_void_p, c_void_p,
         ]
         lib.rl_gemm_f32.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
         lib.rl_sample.argtypes = [
@@ -187,9 +188,10 @@ def embedding(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, fault: 
 
 
 def embedding_sum(out: torch.Tensor, stream: torch.Tensor | None, table: torch.Tensor, pair_table: torch.Tensor,
-                  position_table: torch.Tensor, batch, last_token: torch.Tensor, *, mul_prev: int, mul_cur: int) -> torch.Tensor:
-    """``out[t] = table[id_t] + pair_table[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets] + position_table[p_t]``
-    as a float32 sum (also stored to ``stream`` if given); ``pair_table`` has ``buckets + 1`` rows and a request's first
+                  position_table: torch.Tensor | None, batch, last_token: torch.Tensor, *, mul_prev: int, mul_cur: int,
+                  scale: float = 1.0) -> torch.Tensor:
+    """``out[t] = scale * table[id_t] + pair_table[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets] + position_table[p_t]``
+    as a float32 sum (also stored to ``stream`` if given; no position row without a ``position_table``); ``pair_table`` has ``buckets + 1`` rows and a request's first
     token takes the last.  The id before an entry's first row is the one its slot keeps in ``last_token``
     (int32 ``[slots, 1]``), brought up to date here."""
     _need_cuda(out, stream, table, pair_table, position_table, last_token)
@@ -198,8 +200,8 @@ def embedding_sum(out: torch.Tensor, stream: torch.Tensor | None, table: torch.T
                          ("position_table", position_table), ("last_token", last_token)):
         _contig(name, tensor)
     rows, hidden = out.shape
-    if (table.dtype != out.dtype or pair_table.dtype != out.dtype or position_table.dtype != out.dtype
-            or table.shape[1] != hidden or pair_table.shape[1] != hidden or position_table.shape[1] != hidden
+    if (table.dtype != out.dtype or pair_table.dtype != out.dtype or table.shape[1] != hidden or pair_table.shape[1] != hidden
+            or (position_table is not None and (position_table.dtype != out.dtype or position_table.shape[1] != hidden))
             or rows != batch.token_ids.numel() or (stream is not None and stream.shape != out.shape)
             or last_token.numel() != last_token.shape[0] or pair_table.shape[0] < 2):
         raise KernelError("embedding_sum: shapes or dtypes do not agree")
@@ -208,8 +210,8 @@ def embedding_sum(out: torch.Tensor, stream: torch.Tensor | None, table: torch.T
         dtype_tag(out.dtype), _ptr(out), _ptr(stream), _ptr(table), _ptr(pair_table), _ptr(position_table),
         _ptr(batch.token_ids), _ptr(feedback), 0 if feedback is None else feedback.numel(), _ptr(batch.positions),
         _ptr(batch.cu_seqlens), _ptr(batch.entry_slot), batch.num_entries, _ptr(last_token), last_token.shape[0], rows,
-        hidden, table.shape[0], pair_table.shape[0] - 1, int(mul_prev), int(mul_cur), position_table.shape[0],
-        _ptr(batch.fault), _stream()), "embedding_sum")
+        hidden, table.shape[0], pair_table.shape[0] - 1, int(mul_prev), int(mul_cur),
+        0 if position_table is None else position_table.shape[0], float(scale), _ptr(batch.fault), _stream()), "embedding_sum")
     return out
 
 
@@ -473,13 +475,15 @@ def qk_norm_rope_write(
     cache: torch.Tensor | None = None,
     page_size: int = 1,
     norm_size: int | None = None,
+    temperature: tuple[float, float] | None = None,
 ) -> torch.Tensor:
     """Per-head q/k RMSNorm, rotation by position, q to ``q_out``, k and v into the pages.
 
     ``norm_size``: entries of a head the norm's mean is taken over, when the head's tail is padding.
+    ``temperature = (coef, every)`` multiplies the query at position ``p`` by ``1 + coef ln(floor((p + 1) / every) + 1)``.
 
     ``qkv`` is ``[T, (Hq + 2 Hkv) D]`` (or ``[T, Hq D]`` when ``kv_dest`` is ``None`` and
-    only queries are produced).  ``cache`` is one layer's ``[pages, 2, Hkv, page, D]``;
+    only queries are produced); columns behind those belong to somebody else.  ``cache`` is one layer's ``[pages, 2, Hkv, page, D]``;
     ``kv_dest[t] = page * page_size + offset``.
     """
     _need_cuda(qkv, q_out, cos, sin, positions, fault, q_weight, k_weight, bias, kv_dest, cache)
@@ -490,8 +494,11 @@ def qk_norm_rope_write(
     _expect("positions", positions, torch.int32), _expect("kv_dest", kv_dest, torch.int32)
     tokens, row_width = qkv.shape
     heads_in = num_heads + 2 * num_kv_heads if kv_dest is not None else num_heads
-    if row_width != heads_in * head_dim:
-        raise KernelError(f"qk_norm_rope_write: qkv width {row_width} is not {heads_in} heads of {head_dim}")
+    if row_width < heads_in * head_dim:
+        raise KernelError(f"qk_norm_rope_write: qkv width {row_width} is less than {heads_in} heads of {head_dim}")
+    coef, every = temperature or (0.0, 0.0)
+    if temperature is not None and not every > 0:
+        raise KernelError("qk_norm_rope_write: the temperature's `every` must be positive")
     if q_out.numel() != tokens * num_heads * head_dim or q_out.dtype != qkv.dtype:
         raise KernelError("qk_norm_rope_write: q_out does not fit")
     if cos.shape != sin.shape or cos.dim() != 2 or cos.shape[1] * 2 != rotary_dim:
@@ -506,7 +513,7 @@ def qk_norm_rope_write(
             dtype_tag(qkv.dtype), _ptr(qkv), row_width, _ptr(bias), _ptr(q_weight), _ptr(k_weight),
             _ptr(cos), _ptr(sin), _ptr(positions), _ptr(kv_dest), _ptr(q_out), _ptr(cache), tokens,
             num_heads, num_kv_heads, head_dim, rotary_dim, cos.shape[0], page_size, num_pages,
-            float(eps), int(norm_size or 0), _ptr(fault), int(PDL), _stream(),
+            float(eps), int(norm_size or 0), float(coef), float(every), _ptr(fault), int(PDL), _stream(),
         ),
         f"qk_norm_rope_write(head_dim={head_dim})",
     )
@@ -531,16 +538,16 @@ def attention_generic(
     sink: torch.Tensor | None = None,
     chunk: int = 0,
     gate: torch.Tensor | None = None,
+    slopes: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """Causal attention of every token of the step over its request's cached keys: all of them, the last ``window``
     positions, or (``chunk`` > 0) those of the position's own chunk, counted from position 0.  ``softcap`` > 0 squashes the
     scaled scores to ``softcap * tanh(s / softcap)``; ``sink`` (float32 ``[heads]``) adds ``exp(sink[h])`` to every
-    row's denominator; ``gate`` (``[T, heads]``) multiplies a head's output by its sigmoid.  ``out`` (rows) and ``gate``
+    row's denominator; ``slopes`` (float32 ``[heads]``) takes ``slopes[h] * (query position - key position)`` off every
+    score; ``gate`` (``[T, heads]``) multiplies a head's output by its sigmoid.  ``out`` (rows) and ``gate``
     may be views of some columns of wider rows."""
-    _need_cuda(q, cache, out, positions, token_slot, block_table, fault, sink, gate)
-    _expect("sink", sink, torch.float32), _contig("sink", sink)
-    if sink is not None and sink.numel() != num_heads:
-        raise KernelError("attention: one sink per head")
+    _need_cuda(q, cache, out, positions, token_slot, block_table, fault, sink, gate, slopes)
+    _per_head(num_heads, sink=sink, slopes=slopes)
     _contig("q", q), _contig("cache", cache), _contig("block_table", block_table)
     for name, tensor in (("positions", positions), ("token_slot", token_slot), ("block_table", block_table)):
         _expect(name, tensor, torch.int32)
@@ -559,11 +566,18 @@ def attention_generic(
             dtype_tag(q.dtype), _ptr(q), _ptr(cache), _ptr(out), out_stride, _ptr(gate), gate_stride, _ptr(positions), _ptr(token_slot),
             _ptr(block_table), tokens, num_heads, num_kv_heads, head_dim, cache.shape[3],
             cache.shape[0], block_table.shape[1], block_table.shape[0], int(window), int(chunk), float(scale),
-            float(softcap), _ptr(sink), int(cache.shape[1]), _ptr(fault), _stream(),
+            float(softcap), _ptr(sink), _ptr(slopes), int(cache.shape[1]), _ptr(fault), _stream(),
         ),
         f"attention_generic(head_dim={head_dim})",
     )
     return out
+
+
+def _per_head(num_heads: int, **vectors: torch.Tensor | None) -> None:
+    for name, tensor in vectors.items():
+        _expect(name, tensor, torch.float32), _contig(name, tensor)
+        if tensor is not None and tensor.numel() != num_heads:
+            raise KernelError(f"attention: {name} holds one number per head")
 
 
 def _attention_out(out: torch.Tensor, gate: torch.Tensor | None, tokens: int, num_heads: int, head_dim: int) -> tuple[int, int]:
@@ -605,8 +619,8 @@ def attention_lib(head_dim: int) -> ctypes.CDLL:
         lib.rl_attention_mma.argtypes = [
             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-            c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int,
-            c_int, c_void_p, c_int, c_void_p,
+            c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
+            c_int, c_int, c_void_p, c_int, c_void_p,
         ]
         lib.rl_attention_mma.restype = c_int
         lib.rl_attention_decode_max_clusters.argtypes = [c_int]
@@ -665,6 +679,7 @@ def attention_mma(
     sink: torch.Tensor | None = None,
     chunk: int = 0,
     gate: torch.Tensor | None = None,
+    slopes: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """bfloat16 paged causal attention over work items the host cut the step into.
 
@@ -687,13 +702,12 @@ def attention_mma(
     tiles run on mma.sync (and have no split count of their own).  A position sees all keys up to its own, or the last
     ``window`` of them, or (``chunk`` > 0) those of its own chunk, chunks being counted from position 0.  ``gate``
     (``[T, heads]``) multiplies a head's output by its sigmoid.  ``out`` and ``gate`` may be views of some columns of
-    wider rows.
+    wider rows.  ``slopes`` (float32 ``[heads]``, caches of two planes) takes ``slopes[h] * (query position - key position)``
+    off every score (after a cap).
     """
     _need_cuda(q, cache, out, chunk_items, decode_items, part_out, part_lse, cu_seqlens, entry_start,
-               entry_slot, block_table, fault, sink, gate)
-    _expect("sink", sink, torch.float32), _contig("sink", sink)
-    if sink is not None and sink.numel() != num_heads:
-        raise KernelError("attention: one sink per head")
+               entry_slot, block_table, fault, sink, gate, slopes)
+    _per_head(num_heads, sink=sink, slopes=slopes)
     for name, tensor in (("q", q), ("cache", cache), ("out", out)):
         _expect(name, tensor, torch.bfloat16)
     _contig("q", q), _contig("cache", cache)
@@ -723,7 +737,7 @@ def attention_mma(
             _ptr(block_table), tokens, num_heads, num_kv_heads, head_dim, cache.shape[3], cache.shape[0],
             block_table.shape[1], block_table.shape[0], int(window), int(chunk), int(splits), float(scale),
             _ptr(fault), int(PDL), {"auto": 0, "mma": 1, "deep": 2, "shallow": 3}[decode_kernel], int(decode_rows), int(chunk_rows),
-            int(decode_splits), float(softcap), _ptr(sink), int(cache.shape[1]), out_stride, _ptr(gate), gate_stride, _stream(),
+            int(decode_splits), float(softcap), _ptr(sink), _ptr(slopes), int(cache.shape[1]), out_stride, _ptr(gate), gate_stride, _stream(),
         ),
         f"attention_mma(head_dim={head_dim})",
     )
@@ -1090,6 +1104,8 @@ def recurrent() -> ctypes.CDLL:
             c_int, c_int, c_void_p, c_int, c_void_p,
         ]
         lib.rl_exp_decay.argtypes = [c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
+        lib.rl_low_rank_decay.argtypes = [c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_float, c_void_p,
+                                          c_int, c_void_p, c_int, c_int, c_void_p]
         lib.rl_tanh_rows.argtypes = [c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p]
         lib.rl_shift_mix.argtypes = [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_int,
                                      c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p]
@@ -1098,7 +1114,7 @@ def recurrent() -> ctypes.CDLL:
         lib.rl_xielu.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p]
         lib.rl_scaled_sum.argtypes = [c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_longlong, c_int, c_void_p]
         for name in ("rl_causal_conv_silu", "rl_activate_rows", "rl_decay_gate", "rl_unit_heads", "rl_rotate_heads", "rl_linear_scan",
-                     "rl_gated_norm", "rl_xielu", "rl_scaled_sum", "rl_exp_decay", "rl_tanh_rows", "rl_shift_mix"):
+                     "rl_gated_norm", "rl_xielu", "rl_scaled_sum", "rl_exp_decay", "rl_low_rank_decay", "rl_tanh_rows", "rl_shift_mix"):
             getattr(lib, name).restype = c_int
         _RECURRENT_SET = True
     return lib
@@ -1276,6 +1292,31 @@ def exp_decay(x: torch.Tensor, bias: torch.Tensor | None, decay: torch.Tensor) -
     return decay
 
 
+def low_rank_decay(x: torch.Tensor, low: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, tau: float,
+                   rows: torch.Tensor, decay: torch.Tensor) -> torch.Tensor:
+    """``decay = sigmoid(low @ weight^T + bias) ** (1 / tau)`` as float32 ``[T, C]`` from ``low [T, rank]`` and
+    ``weight [C, rank]`` (engine dtype, float32 sums in a fixed order), and ``rows = x`` as float32; ``x`` and ``low`` are
+    columns of one buffer of rows."""
+    _need_cuda(x, low, weight, bias, rows, decay)
+    for name, tensor in (("bias", bias), ("rows", rows), ("decay", decay)):
+        _expect(name, tensor, torch.float32), _contig(name, tensor)
+    _contig("weight", weight)
+    tokens, rank = low.shape
+    channels = weight.shape[0]
+    stride = _row_stride("x", x)
+    if (rows.shape != x.shape or x.shape[0] != tokens or decay.shape != (tokens, channels) or weight.shape[1] != rank
+            or bias.numel() != channels or weight.dtype != x.dtype or low.dtype != x.dtype or not tau > 0
+            or (tokens > 1 and low.stride(0) != stride) or rank < 1 or low.data_ptr() < x.data_ptr()):
+        raise KernelError("low_rank_decay: shapes or dtypes do not agree")
+    low_col0 = (low.data_ptr() - x.data_ptr()) // x.element_size()
+    if low_col0 + rank > stride:
+        raise KernelError("low_rank_decay: x and low must be columns of the same rows")
+    _check(recurrent().rl_low_rank_decay(
+        dtype_tag(x.dtype), _ptr(x), stride, x.shape[1], int(low_col0), _ptr(weight), rank, _ptr(bias), float(tau), _ptr(rows),
+        channels, _ptr(decay), tokens, int(PDL), _stream()), "low_rank_decay")
+    return decay
+
+
 def tanh_rows(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """``out = tanh(x)`` (float32 arithmetic, one rounding), both contiguous and of one dtype; may be in place."""
     _need_cuda(x, out)
@@ -1329,26 +1370,28 @@ def latent_lib() -> ctypes.CDLL:
 
 
 def latent_norm_write(down: torch.Tensor, *, q_col0: int, q_rank: int, c_col0: int, kv_rank: int, rot: int,
-                      q_weight: torch.Tensor, c_weight: torch.Tensor, eps: float, q_out: torch.Tensor, cache: torch.Tensor,
-                      kv_dest: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor | None, magnitude: float,
+                      q_weight: torch.Tensor, c_weight: torch.Tensor | None, eps: float, q_out: torch.Tensor,
+                      cache: torch.Tensor | None, kv_dest: torch.Tensor | None, positions: torch.Tensor, freq: torch.Tensor | None, magnitude: float,
                       layout: int, fault: torch.Tensor) -> None:
     """From a row ``down[t]`` that holds a query latent (``q_rank`` numbers at ``q_col0``) and ``[c | key part]``
     (``kv_rank + rot`` numbers at ``c_col0``): ``q_out[t]`` = RMS norm of the query latent times ``q_weight``; the
     cache row ``kv_dest[t]`` of ``cache [pages, page_size, D]`` = ``[RMS norm of c times c_weight | the key part
-    rotated by the position | zeros]``.  float32 arithmetic, one rounding."""
+    rotated by the position | zeros]``.  Without a ``cache`` only the query latent is normed (a layer that reads another
+    one's rows).  float32 arithmetic, one rounding."""
     _need_cuda(down, q_weight, c_weight, q_out, cache, kv_dest, positions, freq, fault)
     _expect("q_weight", q_weight, torch.float32), _expect("c_weight", c_weight, torch.float32), _expect("freq", freq, torch.float32)
     _expect("kv_dest", kv_dest, torch.int32), _expect("positions", positions, torch.int32)
     _contig("q_out", q_out), _contig("cache", cache), _contig("freq", freq)
-    tokens, width = down.shape[0], cache.shape[-1]
-    if (q_out.shape != (tokens, q_rank) or q_out.dtype != down.dtype or cache.dtype != down.dtype
-            or q_weight.numel() != q_rank or c_weight.numel() != kv_rank or (rot and freq.numel() != rot // 2)
-            or q_col0 + q_rank > down.shape[1] or c_col0 + kv_rank + rot > down.shape[1] or kv_dest.numel() != tokens):
+    tokens, width = down.shape[0], kv_rank + rot if cache is None else cache.shape[-1]
+    if (q_out.shape != (tokens, q_rank) or q_out.dtype != down.dtype or q_weight.numel() != q_rank
+            or (rot and freq.numel() != rot // 2) or q_col0 + q_rank > down.shape[1]
+            or (cache is not None and (cache.dtype != down.dtype or c_weight is None or c_weight.numel() != kv_rank
+                                       or c_col0 + kv_rank + rot > down.shape[1] or kv_dest is None or kv_dest.numel() != tokens))):
         raise KernelError("latent_norm_write: shapes or dtypes do not agree")
     _check(latent_lib().rl_latent_norm_write(
         dtype_tag(down.dtype), _ptr(down), _row_stride("down", down), int(q_col0), int(q_rank), int(c_col0), int(kv_rank),
         int(rot), _ptr(q_weight), _ptr(c_weight), float(eps), _ptr(q_out), _ptr(cache), _ptr(kv_dest),
-        cache.numel() // width, width, _ptr(positions), _ptr(freq), float(magnitude), int(layout), tokens, _ptr(fault),
+        0 if cache is None else cache.numel() // width, width, _ptr(positions), _ptr(freq), float(magnitude), int(layout), tokens, _ptr(fault),
         int(PDL), _stream()), "latent_norm_write")
 
 

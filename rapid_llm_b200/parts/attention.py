@@ -45,6 +45,11 @@ that reader needs.
 its own chunk, and the pages of a chunk go back to the pool once it is passed.  ``gate="sigmoid_head"`` multiplies head
 ``h``'s output by the one number ``sigmoid(W_g x)_h``; ``o_bias`` adds a bias behind the output projection.
 
+Scores without a rotation: ``slopes`` (a number per query head) takes ``slopes[h] * (i - j)`` off the scaled score of query
+``i`` and key ``j``; ``temperature = (coef, every)`` multiplies the query at position ``p``, behind its norm, by
+``1 + coef ln(floor((p + 1) / every) + 1)``; ``sink_score`` is a fixed score that joins every row's denominator as a learned
+``sink`` would (0: one is added).  ``gate_rides`` puts the gate's rows behind q, k and v in the first product's matrix.
+
 The mixer can stand in an arrangement that stacks its sublayers' products (``first_rows`` and what follows it): its first
 product's rows and its last product's columns then lie in the arrangement's matrices, and :meth:`middle` does what is
 between the two on the columns of the stacked product's result.
@@ -109,20 +114,21 @@ class AttentionItems(StepPlanner):
 
     def __init__(self, group: int, num_kv_heads: int, head_dim: int = 0, sms: int = DEFAULT_SMS,
                  decode_clusters: dict[int, int] | None = None, tensor_core: bool = True,
-                 decode_tensor_core: bool = True, chunk: int = 0) -> None:
+                 decode_tensor_core: bool = True, chunk: int = 0, window: int = 0) -> None:
         self.group, self.num_kv_heads, self.head_dim = int(group), int(num_kv_heads), int(head_dim)
         # decode_tensor_core False: the mixer's scores are squashed, which the tcgen05 chunk tiles and the mma.sync tiles
         # compute, the tcgen05 decode tiles not; tensor_core False: mma.sync tiles only.  chunk: the most keys a
         # position sees (0 = all before it), which bounds the key ranges worth having.
         self.tensor_core = bool(tensor_core)
         self.decode_tensor_core = self.tensor_core and bool(decode_tensor_core)
-        self.chunk = int(chunk)
+        # window: the same bound for the key ranges where a mixer asks for it (0 = not bounded).
+        self.chunk, self.window = int(chunk), int(window)
         self.decode_clusters = dict(decode_clusters or DEFAULT_DECODE_CLUSTERS)
         # work items the kernels want in flight: two CTAs per multiprocessor, one in a decode-only
         # step, whose kernel keeps a whole multiprocessor's shared memory busy
         self.target_ctas, self.decode_target_ctas = 2 * int(sms), int(sms)
         self.key = ("attention_items", self.group, self.num_kv_heads, self.head_dim, int(sms),
-                    tuple(sorted(self.decode_clusters.items())), self.tensor_core, self.decode_tensor_core, self.chunk)
+                    tuple(sorted(self.decode_clusters.items())), self.tensor_core, self.decode_tensor_core, self.chunk, self.window)
 
     def capacity(self, max_tokens: int, max_entries: int) -> int:
         chunk_tiles = -(-max_tokens * self.group // kernels.CHUNK_TILE_ROWS) + max_entries
@@ -147,6 +153,8 @@ class AttentionItems(StepPlanner):
             splits = max(1, min(MAX_SPLITS, target // max(ctas, 1)))
             if self.chunk:
                 splits = max(1, min(splits, -(-self.chunk // kernels.MMA_KEYS)))
+            if self.window:
+                splits = max(1, min(splits, -(-self.window // kernels.MMA_KEYS) + 1))
             if not shape.decode_only:
                 longest = int(seen_last.max())
                 splits = max(1, min(splits, longest // MIN_KEYS_PER_SPLIT))
@@ -240,6 +248,10 @@ class GQAAttention(Mixer):
         rotation: str = "halves",
         values_from_keys: bool = False,
         o_bias: bool = False,
+        slopes=None,
+        temperature: tuple[float, float] | None = None,
+        sink_score: float | None = None,
+        gate_rides: bool = False,
         dtype,
         device,
     ) -> None:
@@ -276,6 +288,13 @@ class GQAAttention(Mixer):
             raise ValueError("rotation by neighbours and values taken from the keys belong to the norm over the whole projection")
         if self.keys_are_values and (self.v_dim != self.qk_dim or shares_cache):
             raise ValueError("values taken from the keys have the keys' size and a cache of their own")
+        if sink and sink_score is not None:
+            raise ValueError("a sink is either learned or fixed")
+        if slopes is not None and len(slopes) != num_heads:
+            raise ValueError(f"slopes holds one number per query head, got {len(slopes)} for {num_heads} heads")
+        self.temperature = None if temperature is None else (float(temperature[0]), float(temperature[1]))
+        if self.temperature is not None and (self.float_prelude or self.row_norm or not self.temperature[1] > 0):
+            raise ValueError("a query temperature belongs to the norm per head (or none) and needs a positive `every`")
         if not 0 <= self.conv_width <= 16 or self.softcap < 0:
             raise ValueError("conv_width must lie between 0 and 16, softcap must not be negative")
         self.names = {name: name for name in (
@@ -307,9 +326,9 @@ class GQAAttention(Mixer):
         self.rotary_dim = int(position.params.get("rotary_dim", getattr(self.position, "rotary_dim", self.d)))
 
         kv_rows = 0 if self.shares_cache else (1 if self.keys_are_values else 2) * self.hkv * self.d
-        # With the norm over the whole projection the gate's rows lie behind q, k and v in ONE matrix: one product
+        # With the norm over the whole projection (or where asked to) the gate's rows lie behind q, k and v in ONE matrix: one product
         # reads the mixer's input once for all four, and the kernels behind it take rows wider than they use.
-        self.gate_rides = bool(self.gate) and self.row_norm
+        self.gate_rides = bool(self.gate) and (self.row_norm or (bool(gate_rides) and not self.float_prelude))
         self.qkv_rows = self.hq * self.d + kv_rows
         self.gate_width = 0 if not self.gate else (self.hq if self.gate == "sigmoid_head" else self.hq * self.d)
         riding = -(-self.gate_width // 8) * 8 if self.gate_rides else 0        # rows of 16 bytes, whatever the head count
@@ -327,6 +346,9 @@ class GQAAttention(Mixer):
             self.g = self._riding_gate() if self.gate_rides else self.new_storage((self.gate_width, self.hidden), MATRIX)
         self.taps = self.new_storage((self.qkv_rows, self.conv_width), VECTOR) if self.conv_width > 0 else None
         self.sink = self.new_storage((self.hq,), VECTOR) if self.has_sink else None
+        if sink_score is not None:
+            self.sink = torch.full((self.hq,), float(sink_score), dtype=torch.float32, device=device)
+        self.slopes = None if slopes is None else torch.tensor([float(s) for s in slopes], dtype=torch.float32).to(device)
         self.mix = self.new_storage((1,), VECTOR) if self.value_mix else None
         self.inv_freq = None
         if (self.float_prelude or self.row_norm) and self.rotary_dim > 0:
@@ -565,7 +587,7 @@ class GQAAttention(Mixer):
             q_weight=self.q_norm, k_weight=self.k_norm,
             kv_dest=group.kv_dest if cache.writes else None,
             cache=cache.pages if cache.writes else None,
-            page_size=group.page_size, norm_size=self.qk_dim,
+            page_size=group.page_size, norm_size=self.qk_dim, temperature=self.temperature,
         )
 
     def attend(self, q, pages, out, batch, group, gate=None) -> None:
@@ -586,7 +608,7 @@ class GQAAttention(Mixer):
                 window=self.window, scale=self.scale, fault=batch.fault, decode_rows=plan.get("decode_rows", 0),
                 chunk_rows=plan.get("chunk_rows", kernels.CHUNK_TILE_ROWS),
                 decode_splits=plan.get("decode_splits", 0), softcap=self.softcap, sink=self.sink, chunk=self.chunk,
-                gate=gate,
+                gate=gate, slopes=self.slopes,
             )
             return
         kernels.attention_generic(
@@ -594,5 +616,5 @@ class GQAAttention(Mixer):
             positions=batch.positions, token_slot=batch.token_slot, block_table=group.block_table,
             num_heads=self.hq, num_kv_heads=self.hkv, head_dim=self.d,
             window=self.window, scale=self.scale, fault=batch.fault, softcap=self.softcap, sink=self.sink, chunk=self.chunk,
-            gate=gate,
+            gate=gate, slopes=self.slopes,
         )

@@ -18,7 +18,12 @@ Options: ``rotation`` ``"halves"`` (entry ``i`` pairs with ``i + rot / 2``) or `
 ``2i + 1``); the nested position part gives the frequencies (``rotary_frequencies``, or ``yarn_frequencies`` with its
 magnitude on cosine and sine); ``head_gate`` multiplies head ``h``'s output by ``sigmoid(W_g x)_h``, one number per
 head from the mixer's input; ``wide_gate`` multiplies the heads side by side, entry by entry, by ``sigmoid(W_g x)``
-(``heads * value_dim`` numbers from the mixer's input).  With ``q_rank=None`` there is no query latent: ``q = W_q x``
+(``heads * value_dim`` numbers from the mixer's input); ``window`` (0 = all keys) lets position ``i`` see the last so many
+positions, its own included, and the pages behind it go back to the pool; ``sink`` adds one learned term
+``exp(sink[head])`` to every row's denominator.  With ``shares_cache`` the layer has no ``W_dkv``: it reads the rows that
+another layer cached (``cache_from`` in the run order) with queries, ``W_uk``, ``W_uv``, window and sink of its own;
+``cache_window`` says how many positions a layer must keep for its readers where that differs from its own window (0 =
+everything).  With ``q_rank=None`` there is no query latent: ``q = W_q x``
 directly (tensor ``q``).  Norms, rotation and the gates are float32; the softmax is float32 in the attention kernels.
 """
 
@@ -38,11 +43,12 @@ def _up8(count: int) -> int:
 
 @MIXERS.register("latent_attention")
 class LatentAttention(Mixer):
-    DEFAULT_NAMES = ("dq", "dq.norm", "uq", "q", "dkv", "dkv.norm", "uk", "uv", "g", "o")
+    DEFAULT_NAMES = ("dq", "dq.norm", "uq", "q", "dkv", "dkv.norm", "uk", "uv", "g", "o", "sink")
 
     def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int,
                  q_rank: int | None, scale: float, norm_eps: float, position: PartSpec, rotation: str = "halves",
-                 head_gate: bool = False, wide_gate: bool = False, names: dict[str, str] | None = None, dtype, device) -> None:
+                 head_gate: bool = False, wide_gate: bool = False, window: int = 0, cache_window: int | None = None,
+                 sink: bool = False, shares_cache: bool = False, names: dict[str, str] | None = None, dtype, device) -> None:
         super().__init__(dtype=dtype, device=device)
         if rotation not in ("halves", "neighbours"):
             raise ValueError(f"rotation must be 'halves' or 'neighbours', got {rotation!r}")
@@ -57,6 +63,10 @@ class LatentAttention(Mixer):
             raise ValueError("latent attention: a gate per head or a gate per entry, not both")
         if min(self.h, self.dim, self.vdim, self.kv_rank, 1 if self.direct_q else self.q_rank) < 1 or self.rot < 0 or self.rot % 2:
             raise ValueError("latent attention: sizes must be positive and the rotated size even")
+        self.window, self.shares_cache = int(window), bool(shares_cache)
+        self.cache_window = self.window if cache_window is None else int(cache_window)
+        if self.window < 0 or (self.cache_window and (self.window == 0 or self.cache_window < self.window)):
+            raise ValueError(f"cache_window ({cache_window}) must cover the layer's own window ({window})")
         self.d = -(-(self.kv_rank + self.rot) // 16) * 16          # a cached row, and a query as the attention sees it
         # the tensor-core tiles take rows of up to 256 numbers; wider rows (up to 640) run the one-warp-per-row kernel
         # in either precision
@@ -76,11 +86,14 @@ class LatentAttention(Mixer):
         # one product from the mixer's input: the query latent, [c | k_r], and the heads' gates, each from a column
         # that is a multiple of 8
         self.c_col0 = _up8(self.q_rank)
-        self.g_col0 = self.c_col0 + _up8(self.kv_rank + self.rot)
+        self.g_col0 = self.c_col0 + (0 if self.shares_cache else _up8(self.kv_rank + self.rot))
         self.down_rows = self.g_col0 + (_up8(self.h) if self.has_gate else self.h * self.vdim if self.wide_gate else 0)
+        if self.down_rows == 0:
+            raise ValueError("latent attention that reads another layer's rows needs a query latent of its own")
         self.down = self.new_storage((self.down_rows, self.hidden), MATRIX)
         self.q_norm = self.new_storage((self.q_rank,), VECTOR)
-        self.c_norm = self.new_storage((self.kv_rank,), VECTOR)
+        self.c_norm = None if self.shares_cache else self.new_storage((self.kv_rank,), VECTOR)
+        self.sink = self.new_storage((self.h,), VECTOR) if sink else None
         self.uq = self.new_storage((self.h * (self.dim + self.rot), self.hidden if self.direct_q else self.q_rank), MATRIX)
         self.g = self.down[self.g_col0 :] if self.wide_gate else None      # the wide gate's rows, behind the latent's
         self.uk_t = self.new_storage((self.h, self.kv_rank, self.dim), MATRIX)      # W_uk_h^T: plain query -> latent
@@ -89,10 +102,12 @@ class LatentAttention(Mixer):
         device = torch.device(device)
         sms = torch.cuda.get_device_properties(device).multi_processor_count if device.type == "cuda" else DEFAULT_SMS
         # the mma.sync tiles read a cache of one plane; the tcgen05 tiles do not
-        self._items = AttentionItems(self.h, 1, self.d, sms, None, tensor_core=False)
+        self._items = AttentionItems(self.h, 1, self.d, sms, None, tensor_core=False, window=self.window)
 
     # -- needs ----------------------------------------------------------------- #
     def cache_need(self) -> CacheNeed:
+        if self.cache_window:
+            return CacheNeed("window", window=self.cache_window, token_shape=(self.d,))
         return CacheNeed("full", token_shape=(self.d,))
 
     def step_planner(self) -> StepPlanner | None:
@@ -120,6 +135,10 @@ class LatentAttention(Mixer):
         if self.direct_q:
             del specs["dq"], specs["dq.norm"], specs["uq"]
             specs["q"] = TensorSpec((self.h * (self.dim + self.rot), self.hidden))
+        if self.shares_cache:
+            del specs["dkv"], specs["dkv.norm"]
+        if self.sink is not None:
+            specs["sink"] = TensorSpec((self.h,), VECTOR)
         if self.has_gate:
             specs["g"] = TensorSpec((self.h, self.hidden))
         if self.wide_gate:
@@ -130,7 +149,9 @@ class LatentAttention(Mixer):
         name = self._ours.get(name, "")
         if name == "dq":
             self.down[: self.q_rank].copy_(tensor)
-        elif name == "dkv":
+        elif name == "sink" and self.sink is not None:
+            self.sink.copy_(tensor.to(torch.float32))
+        elif name == "dkv" and not self.shares_cache:
             self.down[self.c_col0 : self.c_col0 + self.kv_rank + self.rot].copy_(tensor)
         elif name == "g" and self.has_gate:
             self.down[self.g_col0 : self.g_col0 + self.h].copy_(tensor)
@@ -140,7 +161,7 @@ class LatentAttention(Mixer):
             self.uq.copy_(tensor)
         elif name == "dq.norm":
             self.q_norm.copy_(tensor.to(torch.float32))
-        elif name == "dkv.norm":
+        elif name == "dkv.norm" and not self.shares_cache:
             self.c_norm.copy_(tensor.to(torch.float32))
         elif name == "uq":
             self.uq.copy_(tensor)
@@ -155,7 +176,8 @@ class LatentAttention(Mixer):
 
     def parameter_bytes(self) -> int:
         matrices = (self.down, self.uq, self.uk_t, self.uv, self.o)
-        return sum(m.numel() for m in matrices) * self.down.element_size() + (self.q_rank + self.kv_rank) * 4
+        vectors = self.q_rank + (0 if self.shares_cache else self.kv_rank) + (0 if self.sink is None else self.h)
+        return sum(m.numel() for m in matrices) * self.down.element_size() + vectors * 4
 
     def workspace_elements_per_token(self) -> int:
         return (self.down_rows + self.q_rank + self.h * (self.dim + self.rot) + 2 * self.h * self.d
@@ -163,8 +185,8 @@ class LatentAttention(Mixer):
 
     # -- forward --------------------------------------------------------------- #
     def forward(self, x, batch, cache):
-        if cache.group is None or cache.pages is None or not cache.writes:
-            raise ValueError("latent attention needs a cache group of its own; the engine did not give this layer one")
+        if cache.group is None or cache.pages is None or cache.writes == self.shares_cache:
+            raise ValueError("latent attention: the cache the engine gave this layer does not match its role in the run order")
         group, space, rows = batch.groups[cache.group], batch.workspace, x.shape[0]
         pages = cache.pages                                       # [pages, page_size, D]
         down = gemm.linear(x, self.down, space.get("latent_down", rows, self.down_rows, x.dtype), batch.fault)
@@ -172,8 +194,9 @@ class LatentAttention(Mixer):
         c_q = space.get("latent_cq", rows, self.q_rank, x.dtype)      # no columns without a query latent
         kernels.latent_norm_write(
             down, q_col0=0, q_rank=self.q_rank, c_col0=self.c_col0, kv_rank=self.kv_rank, rot=self.rot,
-            q_weight=self.q_norm, c_weight=self.c_norm, eps=self.eps, q_out=c_q, cache=pages, kv_dest=group.kv_dest,
-            positions=batch.positions, freq=self.freq, magnitude=self.magnitude, layout=self.layout, fault=batch.fault)
+            q_weight=self.q_norm, c_weight=self.c_norm, eps=self.eps, q_out=c_q, cache=None if self.shares_cache else pages,
+            kv_dest=None if self.shares_cache else group.kv_dest, positions=batch.positions, freq=self.freq,
+            magnitude=self.magnitude, layout=self.layout, fault=batch.fault)
         q = gemm.linear(x if self.direct_q else c_q, self.uq, space.get("latent_q", rows, self.uq.shape[0], x.dtype), batch.fault)
         gemm.flush()
         wide = space.get("latent_wide", rows, self.h * self.d, x.dtype)
@@ -204,9 +227,10 @@ class LatentAttention(Mixer):
                 q, pages, out, chunk_items=plan["chunk_items"], decode_items=plan["decode_items"], splits=splits,
                 part_out=part_out, part_lse=part_lse, cu_seqlens=batch.cu_seqlens, entry_start=batch.entry_start,
                 entry_slot=batch.entry_slot, block_table=group.block_table, num_heads=self.h, num_kv_heads=1,
-                head_dim=self.d, window=0, scale=self.scale, fault=batch.fault, decode_kernel="mma",
+                head_dim=self.d, window=self.window, scale=self.scale, fault=batch.fault, sink=self.sink, decode_kernel="mma",
                 decode_rows=plan.get("decode_rows", 0), chunk_rows=kernels.CHUNK_TILE_ROWS)
             return
         kernels.attention_generic(
             q, pages, out, positions=batch.positions, token_slot=batch.token_slot, block_table=group.block_table,
-            num_heads=self.h, num_kv_heads=1, head_dim=self.d, window=0, scale=self.scale, fault=batch.fault)
+            num_heads=self.h, num_kv_heads=1, head_dim=self.d, window=self.window, scale=self.scale, sink=self.sink,
+            fault=batch.fault)

@@ -13,6 +13,8 @@ prompts and single decoded tokens alike:
 * :class:`ShiftedDecay` (``wkv``) — a decay per token, head and key channel computed from the input, every
   projection reading a blend of the token's row with the row before it, and a bonus for the token's own pair:
   ``o = (S + diag(u) k v^T)^T r; S <- diag(w) S + k v^T``.
+* :class:`GatedLinear` (``gated_linear``) — a decay per token, head and key channel, the root of a sigmoid of a
+  low-rank product of the input: ``S <- diag(a) S + k v^T; o = S^T q``.
 * :class:`StateSpaceDual` (``state_space_dual``) — the selective state space in its recurrent form:
   ``S <- exp(-exp(A) dt) S + dt B x^T; y = S^T C + D x``.
 
@@ -505,3 +507,90 @@ class ShiftedDecay(_Recurrent):
         kernels.gated_norm(read, normed, group=self.dim, gate=proj[3 * rows :], act=kernels.GATE_SILU, weight=self.norm,
                            eps=self.eps)
         return gemm.linear(normed, self.o, space.get("wkv_out", rows, self.hidden, x.dtype), batch.fault)
+
+
+@MIXERS.register("gated_linear")
+class GatedLinear(_Recurrent):
+    """Linear attention with a decay per token, head and key channel: ``q = W_q x * key_dim ** -0.5``, ``k = W_k x``,
+    ``v = W_v x``, ``a = sigmoid(W_a2 (W_a1 x) + bias) ** (1 / tau)``; per head ``S <- diag(a) S + k v^T`` and
+    ``o = S^T q``.  Every head's read-out is divided by its root mean square and multiplied by ``norm`` (one weight per
+    value channel, shared by the heads); the heads side by side are multiplied by ``SiLU(W_g x)`` and projected.
+
+    One product of the input gives ``[q | k | v | g | W_a1 x]``; the second half of the low-rank pair, its bias and the
+    decay are one float32 kernel.  The queries' factor is not applied: the only thing that reads ``o`` is the norm, and
+    ``(c o) / sqrt(mean((c o)^2) + eps) = o / sqrt(mean(o^2) + eps / c^2)``, so the norm takes ``eps * key_dim``.
+    """
+
+    DEFAULT_NAMES = ("q", "k", "v", "g", "a1", "a2", "a2.b", "norm", "o")
+
+    def __init__(self, *, hidden_size: int, num_heads: int, key_dim: int, value_dim: int, decay_rank: int, tau: float,
+                 norm_eps: float, names: dict[str, str] | None = None, dtype, device) -> None:
+        super().__init__(dtype=dtype, device=device)
+        self._set_names(names)
+        self.hidden, self.h, self.dim, self.vdim = int(hidden_size), int(num_heads), int(key_dim), int(value_dim)
+        self.rank, self.tau, self.eps = int(decay_rank), float(tau), float(norm_eps)
+        if min(self.h, self.dim, self.vdim, self.rank) < 1 or not self.tau > 0:
+            raise ValueError("gated linear attention: sizes and tau must be positive")
+        self.cq, self.cv = self.h * self.dim, self.h * self.vdim
+        self.state_size, self.tail_size = self.h * self.dim * self.vdim, 0
+        # the gate starts on a column that is a multiple of 8, and so do the low-rank columns behind it
+        self.g_col0 = -(-(2 * self.cq + self.cv) // 8) * 8
+        self.a_col0 = self.g_col0 + -(-self.cv // 8) * 8
+        self.w_in = self.new_storage((self.a_col0 + -(-self.rank // 8) * 8, self.hidden), MATRIX)      # q | k | v | g | a1
+        self.a2 = self.new_storage((self.cq, self.rank), MATRIX)
+        self.a2_bias = self.new_storage((self.cq,), VECTOR)
+        self.norm = self.new_storage((self.vdim,), VECTOR)
+        self.o = self.new_storage((self.hidden, self.cv), MATRIX)
+
+    def _tensors(self):
+        return (self.w_in, self.a2, self.a2_bias, self.norm, self.o)
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        return self._named({
+            "q": TensorSpec((self.cq, self.hidden)),
+            "k": TensorSpec((self.cq, self.hidden)),
+            "v": TensorSpec((self.cv, self.hidden)),
+            "g": TensorSpec((self.cv, self.hidden)),
+            "o": TensorSpec((self.hidden, self.cv)),
+            "norm": TensorSpec((self.vdim,), VECTOR, init="ones_normal"),
+            "a1": TensorSpec((self.rank, self.hidden)),
+            "a2": TensorSpec((self.cq, self.rank)),
+            "a2.b": TensorSpec((self.cq,), VECTOR),
+        })
+
+    def load_tensor(self, name: str, tensor: torch.Tensor) -> None:
+        name = self._ours.get(name, "")
+        rows = {"q": 0, "k": self.cq, "v": 2 * self.cq, "g": self.g_col0, "a1": self.a_col0}
+        if name in rows:
+            self.w_in[rows[name] : rows[name] + tensor.shape[0]].copy_(tensor)
+        elif name == "a2":
+            self.a2.copy_(tensor)
+        elif name == "o":
+            self.o.copy_(tensor)
+        elif name == "a2.b":
+            self.a2_bias.copy_(tensor.to(torch.float32))
+        elif name == "norm":
+            self.norm.copy_(tensor.to(torch.float32))
+        else:
+            raise KeyError(name)
+
+    def workspace_elements_per_token(self) -> int:
+        # the product, the float32 q, k, v, decays and read-out, the normed heads and the result
+        return self.w_in.shape[0] + 2 * (3 * self.cq + 2 * self.cv) + self.cv + self.hidden
+
+    def forward(self, x, batch, cache):
+        rows, space, f32 = x.shape[0], batch.workspace, torch.float32
+        S, _ = self._state_views(cache)
+        cq, cv = self.cq, self.cv
+        proj = gemm.linear(x, self.w_in, space.get("gla_in", rows, self.w_in.shape[0], x.dtype), batch.fault)
+        gemm.flush()
+        qkv, decay = space.get("gla_qkv", rows, 2 * cq + cv, f32), space.get("gla_decay", rows, cq, f32)
+        kernels.low_rank_decay(proj[:, : 2 * cq + cv], proj[:, self.a_col0 : self.a_col0 + self.rank], self.a2, self.a2_bias,
+                               self.tau, qkv, decay)
+        read = space.get("gla_read", rows, cv, f32)
+        kernels.linear_scan(qkv[:, :cq], qkv[:, cq : 2 * cq], qkv[:, 2 * cq :], decay, read, S, batch,
+                            heads=self.h, kv_heads=self.h, dim=self.dim, vdim=self.vdim)
+        normed = space.get("gla_normed", rows, cv, x.dtype)
+        kernels.gated_norm(read, normed, group=self.vdim, gate=proj[:, self.g_col0 : self.g_col0 + cv], act=kernels.GATE_SILU,
+                           weight=self.norm, eps=self.eps * self.dim)
+        return gemm.linear(normed, self.o, space.get("gla_out", rows, self.hidden, x.dtype), batch.fault)

@@ -115,6 +115,15 @@ def checkpoint_files(model_dir: str | Path) -> list[Path]:
     return files
 
 
+def tensor_shapes(model_dir: str | Path) -> dict[str, tuple[int, ...]]:
+    """Every tensor's shape by name, from the headers of a folder's files (nothing else is read)."""
+    shapes: dict[str, tuple[int, ...]] = {}
+    for path in sorted(Path(model_dir).glob("*.safetensors")):
+        with SafetensorsFile(path) as handle:
+            shapes.update({name: tuple(handle.shape(name)) for name in handle.keys()})
+    return shapes
+
+
 def iterate_tensors(model_dir: str | Path) -> Iterator[tuple[str, SafetensorsFile]]:
     """Yield ``(name, file)`` for every tensor of every shard, names sorted per shard."""
     for path in checkpoint_files(model_dir):
