@@ -763,6 +763,34 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanArg
           vv[g] = vj;
           continue;
         }
+        if (a.beta == nullptr) {
+          // nothing of the state enters what is added to it: decay and sum are one multiply-add, the only step that a
+          // token has to wait for the one before it
+          const float uj = sbeta[tt + g] * vj;
+          float even = 0.0f, odd = 0.0f;
+          if (a.decay_mode == 2) {
+#pragma unroll
+            for (int r = 0; r < kRows; r += 4) {
+              const float4 g4 = *reinterpret_cast<const float4*>(gp + g * dim_padded + r);
+              S[r] = fmaf(S[r], g4.x, kk[r] * uj);
+              S[r + 1] = fmaf(S[r + 1], g4.y, kk[r + 1] * uj);
+              S[r + 2] = fmaf(S[r + 2], g4.z, kk[r + 2] * uj);
+              S[r + 3] = fmaf(S[r + 3], g4.w, kk[r + 3] * uj);
+            }
+          } else {
+            const float d = sdecay[tt + g];
+#pragma unroll
+            for (int r = 0; r < kRows; ++r) S[r] = fmaf(S[r], d, kk[r] * uj);
+          }
+#pragma unroll
+          for (int r = 0; r < kRows; r += 2) {
+            even += S[r] * qq[r];
+            odd += S[r + 1] * qq[r + 1];
+          }
+          o[g] = even + odd;
+          vv[g] = vj;
+          continue;
+        }
         if (a.decay_mode == 2) {
 #pragma unroll
           for (int r = 0; r < kRows; r += 4) {
@@ -774,21 +802,16 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanArg
 #pragma unroll
           for (int r = 0; r < kRows; ++r) S[r] *= d;
         }
-        float u;
-        if (a.beta) {
-          float seen = 0.0f, seen_odd = 0.0f;
+        float seen = 0.0f, seen_odd = 0.0f;
 #pragma unroll
-          for (int r = 0; r < kRows; r += 2) {
-            seen += S[r] * kk[r];
-            seen_odd += S[r + 1] * kk[r + 1];
-          }
-          seen += seen_odd;
-#pragma unroll
-          for (int offset = cols_per_warp; offset < 32; offset <<= 1) seen += __shfl_xor_sync(0xffffffffu, seen, offset);
-          u = sbeta[tt + g] * (vj - seen);
-        } else {
-          u = sbeta[tt + g] * vj;
+        for (int r = 0; r < kRows; r += 2) {
+          seen += S[r] * kk[r];
+          seen_odd += S[r + 1] * kk[r + 1];
         }
+        seen += seen_odd;
+#pragma unroll
+        for (int offset = cols_per_warp; offset < 32; offset <<= 1) seen += __shfl_xor_sync(0xffffffffu, seen, offset);
+        const float u = sbeta[tt + g] * (vj - seen);
         float even = 0.0f, odd = 0.0f;
 #pragma unroll
         for (int r = 0; r < kRows; r += 2) {

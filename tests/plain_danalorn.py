@@ -14,8 +14,19 @@ import torch
 F64 = torch.float64
 
 
+_STORE = None      # what rounding() does to a number where an engine stores it; None: nothing
+
+
 def _t(tensors, name):
     return tensors[name].to(F64)
+
+
+def _stored(x: torch.Tensor) -> torch.Tensor:
+    return x if _STORE is None else _STORE(x)
+
+
+def _linear(x: torch.Tensor, tensors, name: str) -> torch.Tensor:
+    return _stored(x @ _t(tensors, name).T)
 
 
 def over_rms(x: torch.Tensor, eps: float) -> torch.Tensor:
@@ -79,9 +90,9 @@ def weights_with_sink(scores: torch.Tensor, seen: torch.Tensor, sink: torch.Tens
 def latent_rows(h, tensors, prefix, sizes, eps):
     """What a layer with a latent of its own caches: ``(c [T, rank], rotated key part [T, rot])``."""
     rank = int(sizes["kv_rank"])
-    down = h @ _t(tensors, prefix + "dkv").T
-    c = rms_norm(down[:, :rank], _t(tensors, prefix + "dkv.norm"), eps)
-    return c, rotate_neighbours(down[:, rank:], float((sizes.get("rot") or {}).get("base", 1.0)))
+    down = _linear(h, tensors, prefix + "dkv")
+    c = _stored(rms_norm(down[:, :rank], _t(tensors, prefix + "dkv.norm"), eps))
+    return c, _stored(rotate_neighbours(down[:, rank:], float((sizes.get("rot") or {}).get("base", 1.0))))
 
 
 def latent_attention(h, tensors, prefix, sizes, eps, source):
@@ -89,15 +100,15 @@ def latent_attention(h, tensors, prefix, sizes, eps, source):
     T = h.shape[0]
     H, dim, rot, vdim = (int(sizes[key]) for key in ("heads", "dim", "rot_dim", "vdim"))
     c, k_rot = source
-    c_q = rms_norm(h @ _t(tensors, prefix + "dq").T, _t(tensors, prefix + "dq.norm"), eps)
-    q = (c_q @ _t(tensors, prefix + "uq").T).view(T, H, dim + rot)
+    c_q = _stored(rms_norm(_linear(h, tensors, prefix + "dq"), _t(tensors, prefix + "dq.norm"), eps))
+    q = _linear(c_q, tensors, prefix + "uq").view(T, H, dim + rot)
     q_rot = rotate_neighbours(q[..., dim:], float((sizes.get("rot") or {}).get("base", 1.0)))
-    k = (c @ _t(tensors, prefix + "uk").T).view(T, H, dim)
-    v = (c @ _t(tensors, prefix + "uv").T).view(T, H, vdim)
+    k = _linear(c, tensors, prefix + "uk").view(T, H, dim)
+    v = _linear(c, tensors, prefix + "uv").view(T, H, vdim)
     scores = torch.einsum("ihd,jhd->hij", q[..., :dim], k) + torch.einsum("ihd,jd->hij", q_rot, k_rot)
     seen = visible(T, int((sizes.get("mask") or {}).get("size", 0)))
     shares = weights_with_sink(scores * float(sizes["scale"]), seen, _t(tensors, prefix + "sink"))
-    return torch.einsum("hij,jhd->ihd", shares, v).reshape(T, H * vdim) @ _t(tensors, prefix + "o").T
+    return _linear(_stored(torch.einsum("hij,jhd->ihd", shares, v).reshape(T, H * vdim)), tensors, prefix + "o")
 
 
 # ------------------------------------------------------------- attention -- #
@@ -114,7 +125,7 @@ def attention(h, tensors, prefix, sizes, eps):
     H, G, dim, vdim = (int(sizes[key]) for key in ("heads", "kv_heads", "dim", "vdim"))
 
     def projected(name, heads, size):
-        return (h @ _t(tensors, prefix + name).T + _t(tensors, prefix + name + ".b")).view(T, heads, size)
+        return _stored(h @ _t(tensors, prefix + name).T + _t(tensors, prefix + name + ".b")).view(T, heads, size)
 
     q = rms_norm(projected("q", H, dim), _t(tensors, prefix + "q.norm"), eps)
     k = rms_norm(projected("k", G, dim), _t(tensors, prefix + "k.norm"), eps)
@@ -122,27 +133,28 @@ def attention(h, tensors, prefix, sizes, eps):
     warm = sizes.get("q_temp")
     if warm:
         q = q * query_temperature(T, float(warm["coef"]), float(warm["every"]))[:, None, None]
+    q, k = _stored(q), _stored(k)
     k, v = k.repeat_interleave(H // G, dim=1), v.repeat_interleave(H // G, dim=1)
     scores = torch.einsum("ihd,jhd->hij", q, k) * float(sizes["scale"])
     behind = (torch.arange(T)[:, None] - torch.arange(T)[None, :]).to(F64)
     scores = scores - torch.tensor(distance_slopes(H), dtype=F64)[:, None, None] * behind
     shares = weights_with_sink(scores, visible(T, 0), torch.zeros(H, dtype=F64))
     out = torch.einsum("hij,jhd->ihd", shares, v).reshape(T, H * vdim)
-    return (out * torch.sigmoid(h @ _t(tensors, prefix + "g").T)) @ _t(tensors, prefix + "o").T
+    return _linear(_stored(_stored(out) * torch.sigmoid(_linear(h, tensors, prefix + "g"))), tensors, prefix + "o")
 
 
 # ------------------------------------------------- gated linear attention -- #
 def channel_decays(h, tensors, prefix, tau: float) -> torch.Tensor:
-    z = (h @ _t(tensors, prefix + "a1").T) @ _t(tensors, prefix + "a2").T + _t(tensors, prefix + "a2.b")
+    z = _linear(h, tensors, prefix + "a1") @ _t(tensors, prefix + "a2").T + _t(tensors, prefix + "a2.b")
     return torch.sigmoid(z) ** (1.0 / tau)
 
 
 def gated_linear_attention(h, tensors, prefix, sizes, eps):
     T = h.shape[0]
     H, dim, vdim = (int(sizes[key]) for key in ("heads", "dim", "vdim"))
-    q = (h @ _t(tensors, prefix + "q").T).view(T, H, dim) / math.sqrt(dim)
-    k = (h @ _t(tensors, prefix + "k").T).view(T, H, dim)
-    v = (h @ _t(tensors, prefix + "v").T).view(T, H, vdim)
+    q = _linear(h, tensors, prefix + "q").view(T, H, dim) / math.sqrt(dim)
+    k = _linear(h, tensors, prefix + "k").view(T, H, dim)
+    v = _linear(h, tensors, prefix + "v").view(T, H, vdim)
     alpha = channel_decays(h, tensors, prefix, float(sizes["tau"])).view(T, H, dim)
     S = torch.zeros(H, dim, vdim, dtype=F64)
     read = []
@@ -150,13 +162,13 @@ def gated_linear_attention(h, tensors, prefix, sizes, eps):
         S = alpha[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
         read.append(torch.einsum("hkv,hk->hv", S, q[t]))
     out = rms_norm(torch.stack(read), _t(tensors, prefix + "norm"), eps).reshape(T, H * vdim)
-    g = h @ _t(tensors, prefix + "g").T
-    return (out * g * torch.sigmoid(g)) @ _t(tensors, prefix + "o").T
+    g = _linear(h, tensors, prefix + "g")
+    return _linear(_stored(out * g * torch.sigmoid(g)), tensors, prefix + "o")
 
 
 # ---------------------------------------------------------- feed-forward -- #
 def squared_relu_feed_forward(h, tensors, prefix):
-    return (h @ _t(tensors, prefix + "up").T).clamp(min=0).square() @ _t(tensors, prefix + "down").T
+    return _linear(_stored(_linear(h, tensors, prefix + "up").clamp(min=0).square()), tensors, prefix + "down")
 
 
 # -------------------------------------------------------------- the model -- #
@@ -167,7 +179,7 @@ def forward(tokens, tensors, config, return_layers: bool = False):
     streams, cached = [], {}
     for index, layer in enumerate(config["layers"]):
         p, sizes = f"l{index}.", layer["mixer"]
-        h = rms_norm(x, _t(tensors, p + "norm1"), eps)
+        h = _stored(rms_norm(x, _t(tensors, p + "norm1"), eps))
         if layer["type"] == "latent_attention":
             source = sizes.get("kv_from")
             if source is None:
@@ -181,11 +193,36 @@ def forward(tokens, tensors, config, return_layers: bool = False):
             raise ValueError(layer["type"])
         x = x + rms_norm(mixed, _t(tensors, p + "norm1b"), eps)
         if layer.get("mlp") is not None:
-            h = rms_norm(x, _t(tensors, p + "norm2"), eps)
+            h = _stored(rms_norm(x, _t(tensors, p + "norm2"), eps))
             x = x + rms_norm(squared_relu_feed_forward(h, tensors, p + "mlp."), _t(tensors, p + "norm2b"), eps)
         streams.append(x)
-    logits = rms_norm(x, _t(tensors, "final.norm"), eps) @ _t(tensors, "head").T
+    logits = _stored(rms_norm(x, _t(tensors, "final.norm"), eps)) @ _t(tensors, "head").T
     return (logits, torch.stack(streams)) if return_layers else logits
+
+
+def rounding(tokens, tensors, config, dtype: torch.dtype, exact: torch.Tensor, draws: int = 8) -> torch.Tensor:
+    """Per row, how far the logits move when every projection, norm and head output passes ``dtype`` where an engine of that
+    precision stores it: the root mean square of the difference as a share of the row's own (means removed), the most of one
+    rounding and ``draws - 1`` random errors of its size.
+
+    A sublayer's result is normed on its way to the stream, so a result near zero (a read-out whose query hardly meets the
+    state, a squared relu with nothing left of its few entries) comes out as large as any other, with a direction that
+    rounding decides; a row of that kind says little about an engine in 16 bits."""
+    global _STORE
+    size = (exact - exact.mean(-1, keepdim=True)).square().mean(-1).sqrt()
+    generator = torch.Generator().manual_seed(len(tokens))
+    most = torch.zeros_like(size)
+    for draw in range(draws):
+        if draw == 0:
+            _STORE = lambda x: x.to(dtype).to(F64)      # noqa: E731
+        else:
+            _STORE = lambda x: x * (1.0 + (torch.rand(x.shape, generator=generator, dtype=F64) - 0.5) * torch.finfo(dtype).eps)      # noqa: E731
+        try:
+            moved = forward(tokens, tensors, config) - exact
+        finally:
+            _STORE = None
+        most = torch.maximum(most, (moved - moved.mean(-1, keepdim=True)).square().mean(-1).sqrt() / size)
+    return most
 
 
 def greedy(tokens, tensors, config, steps: int) -> list[int]:
