@@ -269,13 +269,13 @@ __global__ void exp_decay_kernel(const T* x, int x_stride, int col0, const float
 // y dimension); a decay's weight row is read once for its tokens.
 constexpr int kDecayThreads = 128;
 constexpr int kDecayTokens = 8;
-constexpr int kDecayRankStep = 32;      // numbers of a weight row held in registers at a time
+constexpr int kDecayRankStep = 16;      // numbers of a weight row held in registers at a time
 
 template <typename T>
 __global__ void __launch_bounds__(kDecayThreads) low_rank_decay_kernel(
     const T* x, int x_stride, int copied, int low_col0, const T* __restrict__ w, int rank, const float* __restrict__ bias,
     float inv_tau, float* rows, int channels, float* decay, int tokens, int decay_blocks, int vector_rows) {
-  __shared__ float low[kDecayTokens][kDecayRankStep];
+  __shared__ __align__(16) float low[kDecayTokens][kDecayRankStep];
   pdl_trigger();
   const int t0 = blockIdx.x * kDecayTokens, count = min(kDecayTokens, tokens - t0);
   if (static_cast<int>(blockIdx.y) >= decay_blocks) {
@@ -346,7 +346,13 @@ __global__ void __launch_bounds__(kDecayThreads) low_rank_decay_kernel(
     for (int i = 0; i < kDecayTokens; ++i) {
       if (i < count) {
 #pragma unroll
-        for (int r = 0; r < kDecayRankStep; ++r) sum[i] = fmaf(wr[r], low[i][r], sum[i]);
+        for (int r = 0; r < kDecayRankStep; r += 4) {
+          const float4 four = *reinterpret_cast<const float4*>(&low[i][r]);
+          sum[i] = fmaf(wr[r], four.x, sum[i]);
+          sum[i] = fmaf(wr[r + 1], four.y, sum[i]);
+          sum[i] = fmaf(wr[r + 2], four.z, sum[i]);
+          sum[i] = fmaf(wr[r + 3], four.w, sum[i]);
+        }
       }
     }
   }

@@ -115,6 +115,26 @@ def test_norm_per_head_without_rotation_and_with_a_temperature(hq, hkv, d, true_
     assert torch.equal(stored[:, 1], rows[:, hq + hkv :])
 
 
+@pytest.mark.parametrize("rotary", [0, 96])
+def test_every_head_of_an_odd_multiple_of_32_is_written_at_many_tokens(rotary):
+    """Heads of 96 have no form in registers: at tens of thousands of heads a step each still gets a warp of its own."""
+    from rapid_llm_b200.ops import kernels
+
+    tokens, hq, hkv, d, page_size = 10_000, 6, 1, 96, 16
+    g = torch.Generator(device=DEVICE).manual_seed(2)
+    qkv = torch.randn(tokens, (hq + 2 * hkv) * d, generator=g, device=DEVICE).to(torch.bfloat16)
+    table = torch.zeros(64, rotary // 2, device=DEVICE)
+    cache = torch.zeros(tokens // page_size + 1, 2, hkv, page_size, d, dtype=torch.bfloat16, device=DEVICE)
+    q_out, fault = torch.full((tokens, hq * d), 7.0, dtype=torch.bfloat16, device=DEVICE), _word()
+    kernels.qk_norm_rope_write(qkv, q_out, num_heads=hq, num_kv_heads=hkv, head_dim=d, rotary_dim=rotary, cos=table + 1.0, sin=table,
+                               positions=torch.arange(tokens, dtype=torch.int32, device=DEVICE) % 64, eps=1e-6, fault=fault,
+                               kv_dest=page_size + torch.arange(tokens, dtype=torch.int32, device=DEVICE), cache=cache, page_size=page_size)
+    assert int(fault.item()) == 0
+    assert torch.equal(q_out, qkv[:, : hq * d])
+    stored = cache.permute(0, 3, 1, 2, 4).reshape(-1, 2 * d)[page_size : page_size + tokens]
+    assert torch.equal(stored, qkv[:, hq * d :])
+
+
 # -------------------------------------------------------------------------------------- latents -- #
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_a_query_latent_alone_is_normed_without_a_cache(dtype):
